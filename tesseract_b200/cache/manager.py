@@ -11,7 +11,7 @@ holds one state slot whether or not the model has state groups
 (src/engine/recurrent.rs:6-38; groups after src/engine/state.rs:31-132).
 
 Pages are allocated when a request's positions first reach them, returned one by one
-once a sliding window has passed them, and all returned when the request ends; returned
+once a sliding window has passed them (pages of first positions that a need keeps stay), and all returned when the request ends; returned
 pages are handed out again first.  ``admit`` with ``reserve_tokens`` sets aside the
 request's peak need in every group (src/engine/kv.rs:36-51), so an admitted request
 cannot run out; without a reservation pages come on demand and ``extend`` raises
@@ -117,7 +117,7 @@ class CacheManager:
         span = group.need.live_span()
         if span is not None:
             live = -(-(span + self.max_step_tokens) // self.page_size) + 1
-            return min(total, live)
+            return min(total, live + self._pinned_pages(group))
         return total
 
     def bytes_per_token(self) -> int:
@@ -205,7 +205,7 @@ class CacheManager:
                 continue
             first_needed = self._first_needed_page(g, state.length)
             held = state.pages[index]
-            for logical in range(state.first_live[index], first_needed):
+            for logical in range(max(state.first_live[index], self._pinned_pages(g)), first_needed):
                 page = held.pop(logical, None)
                 if page is not None:
                     g.pool.give_back(request, page)
@@ -223,6 +223,10 @@ class CacheManager:
             g.pool.release(request, list(state.pages[index].values()))
             g.tables[state.slot, :] = 0
         self.slots.release(request)
+
+    def _pinned_pages(self, group: _Group) -> int:
+        """Leading pages that stay as long as the request lives (they hold positions that every later query reads)."""
+        return -(-group.need.keep_first // self.page_size)
 
     def _first_needed_page(self, group: _Group, next_position: int) -> int:
         """Lowest logical page that a query at ``next_position`` or later can still read."""

@@ -8,6 +8,10 @@
 //            positions that ends in front of the window (block b if (b + 1) * pool <= p - mask_size + 1);
 //            the averages live in pages of their own (entry b of the request's pooled pages, same page layout), are
 //            walked first, and share the softmax with the window's keys;
+//            A sliding window may also keep the first `keep_first` positions of the sequence: a row sees those of them that
+//            its window has passed, walked first, at their own positions;
+//   bias     with `bias_weight` and `bias_rate` (a number per query head each) the key at distance n = p - j loses
+//            bias_weight * ln(1 + bias_rate * n) of its score;
 //   sink     the softmax denominator has one more entry that carries no value, of score 0
 //            (w_j = exp(s_j) / (1 + sum_j exp(s_j))) or, with `sinks`, of a learned score per query head;
 //   softcap  with softcap > 0 a score s becomes softcap * tanh(s / softcap) (the sink's score is not touched);
@@ -39,31 +43,40 @@ constexpr int kWarps = 4;
 enum MaskKind : int { MASK_CAUSAL = 0, MASK_WINDOW = 1, MASK_BLOCKS = 2, MASK_WINDOW_POOLED = 3 };
 
 // What only some mixers use: a learned sink score per query head (null: none, or the fixed 0 of `sink`), a cap on the
-// scores (0: none), and the pooled blocks of MASK_WINDOW_POOLED (their pages, the requests' tables of those pages and
-// the tokens a block holds).
+// scores (0: none), the pooled blocks of MASK_WINDOW_POOLED (their pages, the requests' tables of those pages and
+// the tokens a block holds), the first positions that MASK_WINDOW keeps, and the distance bias's two numbers per query
+// head (null: none).
 struct MaskExtras {
     const float* sinks;
     float softcap;
     const void* pool_cache;
     const int* pool_table;
     int pool_bt_stride, pool;
+    int keep_first;
+    const float *bias_weight, *bias_rate;
 };
 
 __device__ __forceinline__ float capped(float s, float softcap) {
     return softcap > 0.0f ? softcap * tanhf(s / softcap) : s;
 }
 
-// The keys of a row in the order they are walked: `pooled` averaged blocks, then the positions first_key .. pos.
+// The keys of a row in the order they are walked: `lead` entries in front of the window (averaged blocks, or the kept
+// first positions 0 .. lead - 1), then the positions first_key .. pos.
 struct Reach {
-    int first_key, pooled, total;
-    __device__ Reach(int pos, int mask_kind, int mask_size, int pool) {
+    int first_key, lead, total;
+    bool averages;                // the leading entries are averaged blocks
+    __device__ Reach(int pos, int mask_kind, int mask_size, int pool, int keep_first) {
         first_key = 0;
-        pooled = 0;
+        lead = 0;
+        averages = mask_kind == MASK_WINDOW_POOLED;
         if (mask_kind == MASK_WINDOW || mask_kind == MASK_WINDOW_POOLED) first_key = pos - mask_size + 1 > 0 ? pos - mask_size + 1 : 0;
         else if (mask_kind == MASK_BLOCKS) first_key = (pos / mask_size) * mask_size;
-        if (mask_kind == MASK_WINDOW_POOLED) pooled = first_key / pool;       // blocks that end in front of the window
-        total = pooled + pos - first_key + 1;
+        if (averages) lead = first_key / pool;                                // blocks that end in front of the window
+        else if (mask_kind == MASK_WINDOW) lead = min(keep_first, first_key); // (what the window holds is not walked twice)
+        total = lead + pos - first_key + 1;
     }
+    __device__ bool averaged(int at) const { return averages && at < lead; }
+    __device__ int key(int at) const { return at < lead ? at : first_key + at - lead; }     // position, or block, of entry `at`
 };
 
 // Where a page keeps what.  keys_per_value >= 1: [kv_heads][page][dim] keys, then [kv_heads / keys_per_value][page][vdim]
@@ -105,7 +118,7 @@ attention_masked_kernel(const T* __restrict__ q, int64_t q_stride, const T* __re
     const int kv_head = head / (heads / kv_heads);
     const int pos = positions[row];
     const int seq = seq_of_row[row];
-    const Reach reach(pos, mask_kind, mask_size, extras.pool);
+    const Reach reach(pos, mask_kind, mask_size, extras.pool, extras.keep_first);
 
     float* qs = q_smem + warp * dim;
     const T* qrow = q + (int64_t)row * q_stride + (int64_t)head * dim;
@@ -120,6 +133,8 @@ attention_masked_kernel(const T* __restrict__ q, int64_t q_stride, const T* __re
     const int* pool_table = extras.pool_table == nullptr ? nullptr : extras.pool_table + (int64_t)seq * extras.pool_bt_stride;
     const T* pool_cache = reinterpret_cast<const T*>(extras.pool_cache);
 
+    const bool biased = extras.bias_weight != nullptr;
+    const float bias_weight = biased ? extras.bias_weight[head] : 0.0f, bias_rate = biased ? extras.bias_rate[head] : 0.0f;
     const bool starts = sink || extras.sinks != nullptr;
     float m = starts ? (extras.sinks != nullptr ? extras.sinks[head] : 0.0f) : -1.0e30f;
     float l = starts ? 1.0f : 0.0f;
@@ -133,8 +148,8 @@ attention_masked_kernel(const T* __restrict__ q, int64_t q_stride, const T* __re
         int64_t v_row = 0;                            // the address of the key's value row
         float s = -1.0e30f;
         if (valid) {
-            const bool averaged = at < reach.pooled;
-            const int key = averaged ? at : reach.first_key + at - reach.pooled;
+            const bool averaged = reach.averaged(at);
+            const int key = reach.key(at);
             const T* from = averaged ? pool_cache : cache;
             const int64_t page = (averaged ? pool_table : table)[key / page_size];
             const int in_page = key % page_size;
@@ -153,6 +168,7 @@ attention_masked_kernel(const T* __restrict__ q, int64_t q_stride, const T* __re
                 for (int i = 0; i < dim; ++i) dot = fmaf(qs[i], Elem<T>::load(kp + i), dot);
             }
             s = capped(dot * scale, extras.softcap);
+            if (biased) s -= bias_weight * log1pf(bias_rate * (float)(pos - key));
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float p = valid ? expf(s - m_new) : 0.0f;
@@ -225,7 +241,7 @@ attention_masked_packets_kernel(const T* __restrict__ q, int64_t q_stride, const
     const int kv_head = head0 / (heads / kv_heads);
     const int pos = positions[row];
     const int seq = seq_of_row[row];
-    const Reach reach(pos, mask_kind, mask_size, extras.pool);
+    const Reach reach(pos, mask_kind, mask_size, extras.pool, extras.keep_first);
 
     const T* qrow = q + (int64_t)row * q_stride + (int64_t)head0 * dim;       // the HPW heads lie side by side
     for (int i = lane * N; i < HPW * dim; i += 32 * N) Packet<T>::load(qrow + i, qs + i);
@@ -241,6 +257,7 @@ attention_masked_packets_kernel(const T* __restrict__ q, int64_t q_stride, const
     const int vg = lane / lv, vs = lane % lv;         // value phase: group vg owns keys vg, vg + 32 / lv, ...
     const int value_step = 32 / lv;
 
+    const bool biased = extras.bias_weight != nullptr;
     float m[HPW], l[HPW], acc[HPW][NP][N];
     const bool starts = (sink || extras.sinks != nullptr) && (!SPLIT || warp == 0);       // the sink is the start of one running softmax
 #pragma unroll
@@ -256,8 +273,8 @@ attention_masked_packets_kernel(const T* __restrict__ q, int64_t q_stride, const
     for (int v0 = SPLIT ? 32 * warp : 0; v0 < reach.total; v0 += SPLIT ? 32 * WARPS : 32) {
         const bool valid = v0 + lane < reach.total;
         const int at = valid ? v0 + lane : reach.total - 1;       // (a lane behind the last key points at the last key)
-        const bool averaged = at < reach.pooled;
-        const int k = averaged ? at : reach.first_key + at - reach.pooled;
+        const bool averaged = reach.averaged(at);
+        const int k = reach.key(at);
         const T* from = averaged ? pool_cache : cache;
         const int64_t base = (int64_t)(averaged ? pool_table : table)[k / page_size] * page_elems;
         const int in_page = k % page_size;
@@ -287,7 +304,8 @@ attention_masked_packets_kernel(const T* __restrict__ q, int64_t q_stride, const
         float corr[HPW];
 #pragma unroll
         for (int h = 0; h < HPW; ++h) {
-            const float s = valid ? capped(dot[h] * scale, extras.softcap) : -1.0e30f;
+            float s = valid ? capped(dot[h] * scale, extras.softcap) : -1.0e30f;
+            if (biased && valid) s -= extras.bias_weight[head0 + h] * log1pf(extras.bias_rate[head0 + h] * (float)(pos - k));
             const float m_new = fmaxf(m[h], warp_max(s));
             const float p = valid ? __expf(s - m_new) : 0.0f;
             corr[h] = __expf(m[h] - m_new);
@@ -517,21 +535,26 @@ int launch(const void* q, int64_t q_stride, const void* gate, int64_t gate_strid
 // cache: this layer's pages, laid out as keys_per_value says (PageLayout).  mask_kind: 0 causal, 1 window, 2 blocks,
 // 3 window with pooled blocks (pool_cache: the layer's pages of averaged keys and values, pool_table: the requests'
 // tables of those pages with row stride pool_bt_stride, pool: tokens a block).  sinks: null or float32 [heads];
-// softcap: 0 for none.
+// softcap: 0 for none.  keep_first: first positions that a window (kind 1) keeps; bias_weight, bias_rate: null or float32
+// [heads] (not with pooled blocks).
 TB_EXPORT int tb_attention_masked(const void* q, int64_t q_stride, const void* gate, int64_t gate_stride, void* out,
                                   int64_t out_stride, const void* cache, const int* positions, const int* seq_of_row,
                                   const int* block_table, int bt_stride, int rows, int heads, int kv_heads, int dim,
                                   int vdim, int page_size, int mask_kind, int mask_size, int sink, float scale,
                                   int keys_per_value, int out_f32, const float* sinks, float softcap,
-                                  const void* pool_cache, const int* pool_table, int pool_bt_stride, int pool, int dtype,
-                                  cudaStream_t stream) {
+                                  const void* pool_cache, const int* pool_table, int pool_bt_stride, int pool, int keep_first,
+                                  const float* bias_weight, const float* bias_rate, int dtype, cudaStream_t stream) {
     if (rows == 0) return 0;
+    if (keep_first < 0 || (keep_first > 0 && mask_kind != MASK_WINDOW)) return TB_ERR_BAD_SIZE;
+    if ((bias_weight == nullptr) != (bias_rate == nullptr) || (bias_weight != nullptr && mask_kind == MASK_WINDOW_POOLED))
+        return TB_ERR_BAD_SIZE;
     if (mask_kind == MASK_WINDOW_POOLED && (pool < 1 || pool_cache == nullptr || pool_table == nullptr || keys_per_value != 1))
         return TB_ERR_BAD_SIZE;
     if (softcap < 0.0f) return TB_ERR_BAD_SIZE;
     MaskExtras extras;
     extras.sinks = sinks; extras.softcap = softcap; extras.pool_cache = pool_cache; extras.pool_table = pool_table;
     extras.pool_bt_stride = pool_bt_stride; extras.pool = pool;
+    extras.keep_first = keep_first; extras.bias_weight = bias_weight; extras.bias_rate = bias_rate;
     if (dim < 1 || dim > 1024 || vdim < 1 || vdim > 512) return TB_ERR_BAD_SIZE;
     if (kv_heads < 1 || heads < 1 || heads % kv_heads != 0 || page_size < 1) return TB_ERR_BAD_SIZE;
     if (mask_kind < MASK_CAUSAL || mask_kind > MASK_WINDOW_POOLED) return TB_ERR_BAD_SIZE;

@@ -1,7 +1,8 @@
 // Paged attention on the tensor cores, for prompt portions and (second kernel) for steps of few rows, with 32-bit
 // scores and weights kept to 32-bit accuracy: the masks and page layout of attention_masked.cu (keys and values of separate widths; causal, sliding window or
 // blocks of positions, or a window with averaged blocks in front of it, which are walked first, from pages of their
-// own), its learned sink per query head and its cap on the scores, for bfloat16 queries, keys and values.
+// own), its kept first positions, its learned sink per query head, its cap on the scores and its distance bias, for
+// bfloat16 queries, keys and values.
 //
 //   S = Q K^T      mma.sync m16n8k16 on bfloat16 operands with 32-bit accumulators: the products of two bfloat16
 //                  numbers are exact in 32-bit, so these are the 32-bit scores of the stored queries and keys;
@@ -26,13 +27,17 @@ typedef __nv_bfloat16 bf16;
 // What only some mixers use: a learned sink score per query head (null: none), a cap on the scores (0: none), and the
 // averaged blocks of MASK_WINDOW_POOLED: their pages (laid out like the tokens' with one value head a key head), the
 // requests' tables of those pages and the tokens a block holds.  A row at position p sees the blocks
-// 0 .. first_key(p) / pool - 1, then the tokens first_key(p) .. p.
+// 0 .. first_key(p) / pool - 1, then the tokens first_key(p) .. p.  With MASK_WINDOW and keep_first > 0 the leading
+// entries are the tokens 0 .. min(keep_first, first_key(p)) - 1 themselves.  bias_weight, bias_rate: the distance bias's two
+// numbers per query head (null: none).
 struct Extras {
     const float* sinks;
     float softcap, cap_k;                 // cap_k = 2 log2(e) / softcap (0 without a cap)
     const bf16* pool_cache;
     const int* pool_table;
     int pool_bt_stride, pool;
+    int keep_first;
+    const float *bias_weight, *bias_rate;
 };
 
 // softcap * tanh(s / softcap) as softcap - 2 softcap / (2^(s k) + 1) with k = 2 log2(e) / softcap: one exponential and
@@ -82,7 +87,21 @@ __device__ __forceinline__ int first_key_of(int pos, int mask_kind, int mask_siz
     return 0;
 }
 
-template <int D, int DV>
+// Entries that a row whose window begins at `first_key` sees in front of it: averaged blocks, or kept first positions.
+__device__ __forceinline__ int lead_of(int first_key, int mask_kind, const Extras& x) {
+    if (mask_kind == MASK_WINDOW_POOLED) return first_key / x.pool;
+    if (mask_kind == MASK_WINDOW) return min(x.keep_first, first_key);
+    return 0;
+}
+// weight * log2(1 + rate * distance): the bias with ln(2) folded into its weight
+__device__ __forceinline__ float distance_bias(float weight, float rate, int distance) {
+    float v;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(v) : "f"(fmaf(rate, (float)distance, 1.0f)));
+    return weight * v;
+}
+
+// BIASED: the scores lose their distance bias (a kernel of its own: the others keep their registers).
+template <int D, int DV, bool BIASED>
 __global__ void __launch_bounds__(128)
 attention_prompt_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__ out, int64_t out_stride,
                         const bf16* __restrict__ cache, const int* __restrict__ positions,
@@ -115,8 +134,10 @@ attention_prompt_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __re
     const int head = blockIdx.y, kv_head = head / (heads / kv_heads);
     const int pos_first = positions[r0], pos_last = pos_first + n - 1;        // a sequence's rows stand at consecutive positions
     const int key_lo = first_key_of(pos_first, mask_kind, mask_size);
-    // the keys the block walks: the averaged blocks its last row sees, then the tokens key_lo .. pos_last
-    const int blocks_last = mask_kind == MASK_WINDOW_POOLED ? first_key_of(pos_last, mask_kind, mask_size) / x.pool : 0;
+    // the keys the block walks: what its last row sees in front of its window, then the tokens key_lo .. pos_last (a kept
+    // token that an early row's window still holds is walked twice; every row takes it once, where it belongs)
+    const bool averages = mask_kind == MASK_WINDOW_POOLED;
+    const int blocks_last = lead_of(first_key_of(pos_last, mask_kind, mask_size), mask_kind, x);
     const int span = blocks_last + pos_last - key_lo + 1;
     const int tiles = (span - 1) / KT + 1;
     // keys_per_value key heads in a row read one value head: the page holds kv_heads / keys_per_value of those
@@ -135,8 +156,8 @@ attention_prompt_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __re
         const int at = tile * KT + copy_row;
         const bool there = at < span;
         const int a = there ? at : span - 1;
-        const bool averaged = a < blocks_last;
-        const int k = averaged ? a : key_lo + a - blocks_last;
+        const bool averaged = averages && a < blocks_last;
+        const int k = a < blocks_last ? a : key_lo + a - blocks_last;
         const bf16* from = averaged ? x.pool_cache : cache;
         const int64_t base = (int64_t)(averaged ? pool_table : table)[k / page_size] * page_elems;
         const int in_page = k % page_size;
@@ -180,8 +201,10 @@ attention_prompt_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __re
         pos[r] = pos_first + i0 + g + r * 8;
         there[r] = i0 + g + r * 8 < n;
         first_key[r] = first_key_of(pos[r], mask_kind, mask_size);
-        blocks[r] = mask_kind == MASK_WINDOW_POOLED ? first_key[r] / x.pool : 0;
+        blocks[r] = lead_of(first_key[r], mask_kind, x);
     }
+    const float bias_weight = BIASED ? x.bias_weight[head] * 0.6931471805599453f : 0.0f;
+    const float bias_rate = BIASED ? x.bias_rate[head] : 0.0f;
     float m[2] = {-1.0e30f, -1.0e30f}, l[2] = {0.0f, 0.0f};
     if (x.sinks != nullptr) {                                     // the sink is the start of the running softmax
         m[0] = m[1] = x.sinks[head];
@@ -227,16 +250,30 @@ attention_prompt_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __re
             }
             // scale, mask, and the tile's share of the streaming softmax
             float top[2] = {-1.0e30f, -1.0e30f};
+            if constexpr (BIASED) {
 #pragma unroll
-            for (int j = 0; j < KT / 8; ++j)
+                for (int j = 0; j < KT / 8; ++j)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int r = e >> 1, place = j * 8 + 2 * t + (e & 1), key = key0 + place;
-                    const bool seen = there[r] && (at0 + place < blocks_last ? at0 + place < blocks[r]
-                                                                             : key <= pos[r] && key >= first_key[r]);
-                    s[j][e] = seen ? capped(s[j][e] * scale, x.softcap, x.cap_k) : -1.0e30f;
-                    top[r] = fmaxf(top[r], s[j][e]);
-                }
+                    for (int e = 0; e < 4; ++e) {
+                        const int r = e >> 1, place = j * 8 + 2 * t + (e & 1), token = key0 + place, at = at0 + place;
+                        const bool leads = at < blocks_last;
+                        const bool seen = there[r] && (leads ? at < blocks[r] : token <= pos[r] && token >= first_key[r]);
+                        const float lost = distance_bias(bias_weight, bias_rate, max(pos[r] - (leads ? at : token), 0));
+                        s[j][e] = seen ? capped(s[j][e] * scale, x.softcap, x.cap_k) - lost : -1.0e30f;
+                        top[r] = fmaxf(top[r], s[j][e]);
+                    }
+            } else {
+#pragma unroll
+                for (int j = 0; j < KT / 8; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int r = e >> 1, place = j * 8 + 2 * t + (e & 1), key = key0 + place;
+                        const bool seen = there[r] && (at0 + place < blocks_last ? at0 + place < blocks[r]
+                                                                                 : key <= pos[r] && key >= first_key[r]);
+                        s[j][e] = seen ? capped(s[j][e] * scale, x.softcap, x.cap_k) : -1.0e30f;
+                        top[r] = fmaxf(top[r], s[j][e]);
+                    }
+            }
             float corr[2];
 #pragma unroll
             for (int r = 0; r < 2; ++r) {
@@ -322,8 +359,9 @@ attention_rows_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __rest
     const int row = blockIdx.x, kv_head = blockIdx.y, per = heads / kv_heads;
     const int pos = positions[row], seq = seq_of_row[row];
     const int key_lo = first_key_of(pos, mask_kind, mask_size);
-    // the keys the row sees, in the order they are walked: its averaged blocks, then the tokens key_lo .. pos
-    const int blocks = mask_kind == MASK_WINDOW_POOLED ? key_lo / x.pool : 0;
+    // the keys the row sees, in the order they are walked: what lies in front of its window, then the tokens key_lo .. pos
+    const bool averages = mask_kind == MASK_WINDOW_POOLED;
+    const int blocks = lead_of(key_lo, mask_kind, x);
     const int span = blocks + pos - key_lo + 1;
     const int tiles = (span - 1) / KT + 1;
     // keys_per_value key heads in a row read one value head: the page holds kv_heads / keys_per_value of those
@@ -339,8 +377,8 @@ attention_rows_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __rest
         const int at = tile * KT + copy_row;
         const bool there = at < span;
         const int a = there ? at : span - 1;
-        const bool averaged = a < blocks;
-        const int k = averaged ? a : key_lo + a - blocks;
+        const bool averaged = averages && a < blocks;
+        const int k = a < blocks ? a : key_lo + a - blocks;
         const bf16* from = averaged ? x.pool_cache : cache;
         const int64_t base = (int64_t)(averaged ? pool_table : table)[k / page_size] * page_elems;
         const int in_page = k % page_size;
@@ -383,6 +421,16 @@ attention_rows_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __rest
                 l[r] = t == 0 ? 1.0f : 0.0f;
             }
     }
+    const bool biased = x.bias_weight != nullptr;
+    float bias_weight[2] = {0.0f, 0.0f}, bias_rate[2] = {0.0f, 0.0f};
+    if (biased) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+            if (g + r * 8 < per) {
+                bias_weight[r] = x.bias_weight[kv_head * per + g + r * 8] * 0.6931471805599453f;
+                bias_rate[r] = x.bias_rate[kv_head * per + g + r * 8];
+            }
+    }
     float o[DV / 8][4];
 #pragma unroll
     for (int j = 0; j < DV / 8; ++j)
@@ -419,6 +467,10 @@ attention_rows_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __rest
                 for (int e = 0; e < 4; ++e) {
                     const int at = at0 + j * 8 + 2 * t + (e & 1);
                     s[j][e] = at < span ? capped(s[j][e] * scale, x.softcap, x.cap_k) : -1.0e30f;     // (all of the span is inside the mask)
+                    if (biased && at < span) {
+                        const int key = at < blocks ? at : key_lo + at - blocks;
+                        s[j][e] -= distance_bias(bias_weight[e >> 1], bias_rate[e >> 1], pos - key);
+                    }
                     top[e >> 1] = fmaxf(top[e >> 1], s[j][e]);
                 }
             float corr[2];
@@ -522,7 +574,7 @@ int launch(const void* q, int64_t q_stride, void* out, int64_t out_stride, const
            int page_size, int mask_kind, int mask_size, float scale, int keys_per_value, int out_f32, Extras x,
            cudaStream_t stream) {
     constexpr int smem = 2 * KT * (D * 2 + 16 + DV * 2 + 16);
-    auto kernel = attention_prompt_kernel<D, DV>;
+    auto kernel = x.bias_weight != nullptr ? attention_prompt_kernel<D, DV, true> : attention_prompt_kernel<D, DV, false>;
     if (smem > 40 * 1024) {
         cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (err != cudaSuccess) return (int)err;
@@ -533,6 +585,11 @@ int launch(const void* q, int64_t q_stride, void* out, int64_t out_stride, const
                                          bt_stride, num_seqs, heads, kv_heads, page_size, mask_kind, mask_size, scale,
                                          keys_per_value, out_f32, x);
     return launched == cudaSuccess ? tb_launch_status() : (int)launched;
+}
+
+bool extras_fit(int mask_kind, int keep_first, const float* bias_weight, const float* bias_rate) {
+    if (keep_first < 0 || (keep_first > 0 && mask_kind != MASK_WINDOW)) return false;
+    return (bias_weight == nullptr) == (bias_rate == nullptr) && (bias_weight == nullptr || mask_kind != MASK_WINDOW_POOLED);
 }
 
 }  // namespace
@@ -548,14 +605,17 @@ TB_EXPORT int tb_attention_prompt_mma_supported(int dim, int vdim) {
 // value head g / keys_per_value); row_start: int32 [num_seqs + 1]; the rows of a sequence stand at consecutive
 // positions.  mask_kind: 0 causal, 1 window, 2 blocks, 3 window with averaged blocks (pool_cache: the layer's pages of
 // averages, pool_table: the requests' tables of those pages with row stride pool_bt_stride, pool: tokens a block).
-// sinks: null or float32 [heads]; softcap: 0 for none.
+// sinks: null or float32 [heads]; softcap: 0 for none; keep_first: first positions that a window (kind 1) keeps; bias_weight,
+// bias_rate: null or float32 [heads] (a key at distance n loses bias_weight * ln(1 + bias_rate * n); not with pooled blocks).
 TB_EXPORT int tb_attention_prompt_mma(const void* q, int64_t q_stride, void* out, int64_t out_stride, const void* cache,
                                       const int* positions, const int* row_start, const int* block_table, int bt_stride,
                                       int rows, int num_seqs, int heads, int kv_heads, int dim, int vdim, int page_size,
                                       int mask_kind, int mask_size, float scale, int keys_per_value, int out_f32,
                                       const float* sinks, float softcap, const void* pool_cache, const int* pool_table,
-                                      int pool_bt_stride, int pool, cudaStream_t stream) {
+                                      int pool_bt_stride, int pool, int keep_first, const float* bias_weight,
+                                      const float* bias_rate, cudaStream_t stream) {
     if (rows == 0) return 0;
+    if (!extras_fit(mask_kind, keep_first, bias_weight, bias_rate)) return TB_ERR_BAD_SIZE;
     if (mask_kind == MASK_WINDOW_POOLED && (pool < 1 || pool_cache == nullptr || pool_table == nullptr || keys_per_value != 1 ||
                                             (uintptr_t)pool_cache % 16 != 0))
         return TB_ERR_BAD_SIZE;
@@ -563,6 +623,7 @@ TB_EXPORT int tb_attention_prompt_mma(const void* q, int64_t q_stride, void* out
     Extras x;
     x.sinks = sinks; x.softcap = softcap; x.cap_k = softcap > 0.0f ? 2.8853900817779268f / softcap : 0.0f; x.pool_cache = (const bf16*)pool_cache; x.pool_table = pool_table;
     x.pool_bt_stride = pool_bt_stride; x.pool = pool;
+    x.keep_first = keep_first; x.bias_weight = bias_weight; x.bias_rate = bias_rate;
     if (!tb_attention_prompt_mma_supported(dim, vdim)) return TB_ERR_BAD_SIZE;
     if (kv_heads < 1 || heads < 1 || heads % kv_heads != 0 || page_size < 1 || num_seqs < 1) return TB_ERR_BAD_SIZE;
     if (keys_per_value < 1 || kv_heads % keys_per_value != 0) return TB_ERR_BAD_SIZE;
@@ -589,8 +650,10 @@ TB_EXPORT int tb_attention_rows_mma(const void* q, int64_t q_stride, void* out, 
                                     int rows, int heads, int kv_heads, int dim, int vdim, int page_size, int mask_kind,
                                     int mask_size, float scale, int keys_per_value, int out_f32, const float* sinks,
                                     float softcap, const void* pool_cache, const int* pool_table, int pool_bt_stride,
-                                    int pool, cudaStream_t stream) {
+                                    int pool, int keep_first, const float* bias_weight, const float* bias_rate,
+                                    cudaStream_t stream) {
     if (rows == 0) return 0;
+    if (!extras_fit(mask_kind, keep_first, bias_weight, bias_rate)) return TB_ERR_BAD_SIZE;
     if (mask_kind == MASK_WINDOW_POOLED && (pool < 1 || pool_cache == nullptr || pool_table == nullptr || keys_per_value != 1 ||
                                             (uintptr_t)pool_cache % 16 != 0))
         return TB_ERR_BAD_SIZE;
@@ -598,6 +661,7 @@ TB_EXPORT int tb_attention_rows_mma(const void* q, int64_t q_stride, void* out, 
     Extras x;
     x.sinks = sinks; x.softcap = softcap; x.cap_k = softcap > 0.0f ? 2.8853900817779268f / softcap : 0.0f; x.pool_cache = (const bf16*)pool_cache; x.pool_table = pool_table;
     x.pool_bt_stride = pool_bt_stride; x.pool = pool;
+    x.keep_first = keep_first; x.bias_weight = bias_weight; x.bias_rate = bias_rate;
     if (!tb_attention_prompt_mma_supported(dim, vdim)) return TB_ERR_BAD_SIZE;
     if (kv_heads < 1 || heads < 1 || heads % kv_heads != 0 || heads / kv_heads > 16 || page_size < 1) return TB_ERR_BAD_SIZE;
     if (keys_per_value < 1 || kv_heads % keys_per_value != 0) return TB_ERR_BAD_SIZE;

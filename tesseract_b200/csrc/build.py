@@ -65,6 +65,8 @@ SOURCES: Dict[str, List[str]] = {
     "latent_rope_cache": [],
     "attention_latent_mma": [],
     "gated_residual": [],
+    "short_conv": [],
+    "rglru": [],
 }
 
 

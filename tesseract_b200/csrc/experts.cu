@@ -7,13 +7,21 @@
 //                      group counts as much as its best expert, only experts of the `keep` best groups can be chosen;
 //                      of those the `top` with the largest scores, largest first (the lowest index wins a tie), weighted
 //                      by their scores over the chosen scores' sum (+ 1e-20), times `weight_scale`.
+//   tb_choose_sigmoid  the `top` largest logits of a row, largest first (the lowest index wins a tie), each weighted by its
+//                      own sigmoid; the row of logits may be longer than the experts (what lies behind them is not the
+//                      router's).
 //   tb_expert_plan     rows * top assignments (row t, slot s -> assignment t * top + s) are grouped by their expert:
 //                      offsets[e] .. offsets[e + 1] of `order` name the assignments of expert e.
 //   tb_expert_linear   out[a, :] = act(W[expert(a)] in[source(a), :]) for every assignment a, a tile of one expert's
 //                      assignments per block; source(a) is a / top (the row itself: the first product of an expert)
 //                      or a (the second).  Every output number is one chain over K that does not depend on which
 //                      other assignments share its tile.
-//   tb_expert_combine  out[t, :] = [base[t, :] +] sum_s weight[t, s] * y[t * top + s, :], slots in order, 32-bit.
+//                      The gated form takes weight rows that alternate (row 2j: gate, row 2j + 1: up): with G, U the two
+//                      sums, both times the assignment's weight if one is given (the expert then reads its row times
+//                      that weight), g = min(G, limit), u = min(max(U, -limit), limit), it stores
+//                      out[a, j] = g * sigmoid(slope * g) * (u + 1), half as many numbers as the weight has rows.
+//   tb_expert_combine  out[t, :] = [base[t, :] * sigmoid(base_gate[t]) +] sum_s weight[t, s] * y[t * top + s, :], slots in
+//                      order, 32-bit; without weights the slots are added as they are, without base_gate so is the base.
 //
 // Nothing here needs the host to know how many rows an expert received: grids are sized for the worst case and
 // blocks without work leave at once, so a step's launches depend on its row count alone.
@@ -158,6 +166,42 @@ choose_grouped_kernel(const float* __restrict__ logits, int* __restrict__ ids, f
     for (int s = lane; s < top; s += 32) my_weights[s] *= factor;
 }
 
+// A warp a row; logits 32-bit, `experts` of a row of `stride` numbers.
+__global__ void __launch_bounds__(kRouteWarps * 32)
+choose_sigmoid_kernel(const float* __restrict__ logits, int64_t stride, int* __restrict__ ids, float* __restrict__ weights,
+                      int rows, int experts, int top) {
+    extern __shared__ __align__(16) float route_smem[];          // per warp: its row's logits
+    pdl_trigger();
+    pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int row = blockIdx.x * kRouteWarps + warp;
+    if (row >= rows) return;
+    float* zs = route_smem + (size_t)warp * experts;
+    for (int e = lane; e < experts; e += 32) zs[e] = logits[(int64_t)row * stride + e];
+    __syncwarp();
+    for (int s = 0; s < top; ++s) {
+        float best = -INFINITY;
+        int where = 0x7fffffff;
+        for (int e = lane; e < experts; e += 32) {
+            const float v = zs[e];
+            if (v > best) { best = v; where = e; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int ow = __shfl_xor_sync(0xffffffffu, where, o);
+            if (ob > best || (ob == best && ow < where)) { best = ob; where = ow; }
+        }
+        if (where == 0x7fffffff) where = 0;                      // (only if every logit is NaN or -inf)
+        if (lane == 0) {
+            ids[(int64_t)row * top + s] = where;
+            weights[(int64_t)row * top + s] = 1.0f / (1.0f + expf(-best));
+            zs[where] = -INFINITY;
+        }
+        __syncwarp();
+    }
+}
+
 // ----------------------------------------------------------------------------- grouping
 
 __global__ void __launch_bounds__(1024)
@@ -194,7 +238,18 @@ expert_plan_kernel(const int* __restrict__ ids, int assignments, int experts, in
 
 // ----------------------------------------------------------------------------- the experts' products
 
-enum ExpertEpilogue : int { EXP_PLAIN = 0, EXP_SQUARED_RELU = 1 };
+enum ExpertEpilogue : int { EXP_PLAIN = 0, EXP_SQUARED_RELU = 1, EXP_GATED_CLAMPED = 2 };
+
+// What the gated form reads: the assignments' weights (or null) and its two constants.
+struct Gating {
+    const float* row_weights;
+    float limit, slope;
+};
+__device__ __forceinline__ float gated_clamped(float g, float u, float weight, const Gating& gating) {
+    g = fminf(g * weight, gating.limit);
+    u = fminf(fmaxf(u * weight, -gating.limit), gating.limit);
+    return g * (1.0f / (1.0f + expf(-gating.slope * g))) * (u + 1.0f);
+}
 
 constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
 
@@ -221,7 +276,7 @@ template <typename T, typename O, int EPI>
 __global__ void __launch_bounds__(256)
 expert_linear_kernel(const T* __restrict__ in, int64_t in_stride, const T* __restrict__ W, O* __restrict__ out,
                      int64_t out_stride, const int* __restrict__ offsets, const int* __restrict__ order, int experts,
-                     int top_div, int N, int K) {
+                     int top_div, int N, int K, Gating gating) {
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[BK][BN + 4];
     __shared__ int rows_of[BM];
@@ -279,16 +334,25 @@ expert_linear_kernel(const T* __restrict__ in, int64_t in_stride, const T* __res
     for (int i = 0; i < TM; ++i) {
         const int a = rows_of[ty * TM + i];
         if (a < 0) continue;
+        if constexpr (EPI == EXP_GATED_CLAMPED) {
+            const float weight = gating.row_weights == nullptr ? 1.0f : gating.row_weights[a];
 #pragma unroll
-        for (int j = 0; j < TN; ++j) {
-            const int n = n0 + tx * TN + j;
-            if (n >= N) continue;
-            float v = acc[i][j];
-            if (EPI == EXP_SQUARED_RELU) {
-                v = fmaxf(v, 0.0f);
-                v *= v;
+            for (int j = 0; j < TN; j += 2) {
+                const int n = n0 + tx * TN + j;
+                if (n < N) Elem<O>::store(out + (int64_t)a * out_stride + n / 2, gated_clamped(acc[i][j], acc[i][j + 1], weight, gating));
             }
-            Elem<O>::store(out + (int64_t)a * out_stride + n, v);
+        } else {
+#pragma unroll
+            for (int j = 0; j < TN; ++j) {
+                const int n = n0 + tx * TN + j;
+                if (n >= N) continue;
+                float v = acc[i][j];
+                if (EPI == EXP_SQUARED_RELU) {
+                    v = fmaxf(v, 0.0f);
+                    v *= v;
+                }
+                Elem<O>::store(out + (int64_t)a * out_stride + n, v);
+            }
         }
     }
 }
@@ -307,7 +371,8 @@ template <typename O, int EPI>
 __global__ void __launch_bounds__(128)
 expert_linear_mma_kernel(const __nv_bfloat16* __restrict__ in, int64_t in_stride, const __nv_bfloat16* __restrict__ W,
                          O* __restrict__ out, int64_t out_stride, const int* __restrict__ offsets,
-                         const int* __restrict__ order, int experts, int top_div, int N, int K) {
+                         const int* __restrict__ order, int experts, int top_div, int N, int K,
+                         Gating gating) {
     __shared__ __align__(16) __nv_bfloat16 As[BM][MK + MPAD];
     __shared__ __align__(16) __nv_bfloat16 Ws[BN][MK + MPAD];
     __shared__ int rows_of[BM];
@@ -369,18 +434,29 @@ expert_linear_mma_kernel(const __nv_bfloat16* __restrict__ in, int64_t in_stride
     for (int half = 0; half < 2; ++half) {
         const int a = rows_of[warp * 16 + g + half * 8];
         if (a < 0) continue;
+        if constexpr (EPI == EXP_GATED_CLAMPED) {
+            const float weight = gating.row_weights == nullptr ? 1.0f : gating.row_weights[a];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
+            for (int j = 0; j < 8; ++j) {
+                const int n = n0 + j * 8 + 2 * t;
+                if (n < N)
+                    Elem<O>::store(out + (int64_t)a * out_stride + n / 2,
+                                   gated_clamped(acc[j][half * 2], acc[j][half * 2 + 1], weight, gating));
+            }
+        } else {
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int n = n0 + j * 8 + 2 * t + e;
-                if (n >= N) continue;
-                float v = acc[j][half * 2 + e];
-                if (EPI == EXP_SQUARED_RELU) {
-                    v = fmaxf(v, 0.0f);
-                    v *= v;
+            for (int j = 0; j < 8; ++j) {
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int n = n0 + j * 8 + 2 * t + e;
+                    if (n >= N) continue;
+                    float v = acc[j][half * 2 + e];
+                    if (EPI == EXP_SQUARED_RELU) {
+                        v = fmaxf(v, 0.0f);
+                        v *= v;
+                    }
+                    Elem<O>::store(out + (int64_t)a * out_stride + n, v);
                 }
-                Elem<O>::store(out + (int64_t)a * out_stride + n, v);
             }
         }
     }
@@ -410,7 +486,8 @@ template <typename O, int EPI>
 __global__ void __launch_bounds__(256)
 expert_linear_pipe_kernel(const __nv_bfloat16* __restrict__ in, int64_t in_stride, const __nv_bfloat16* __restrict__ W,
                           O* __restrict__ out, int64_t out_stride, const int* __restrict__ offsets,
-                          const int* __restrict__ order, int experts, int top_div, int N, int K) {
+                          const int* __restrict__ order, int experts, int top_div, int N, int K,
+                          Gating gating) {
     extern __shared__ __align__(128) unsigned char pipe_smem[];
     __shared__ int rows_of[PM];
     pdl_trigger();
@@ -497,90 +574,89 @@ expert_linear_pipe_kernel(const __nv_bfloat16* __restrict__ in, int64_t in_strid
         for (int half = 0; half < 2; ++half) {
             const int a = rows_of[wm * 32 + i * 16 + g + half * 8];
             if (a < 0) continue;
+            if constexpr (EPI == EXP_GATED_CLAMPED) {
+                const float weight = gating.row_weights == nullptr ? 1.0f : gating.row_weights[a];
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int n = n0 + wn * 32 + j * 8 + 2 * t + e;
-                    if (n >= N) continue;
-                    float v = acc[i][j][half * 2 + e];
-                    if (EPI == EXP_SQUARED_RELU) {
-                        v = fmaxf(v, 0.0f);
-                        v *= v;
-                    }
-                    Elem<O>::store(out + (int64_t)a * out_stride + n, v);
+                for (int j = 0; j < 4; ++j) {
+                    const int n = n0 + wn * 32 + j * 8 + 2 * t;
+                    if (n < N)
+                        Elem<O>::store(out + (int64_t)a * out_stride + n / 2,
+                                       gated_clamped(acc[i][j][half * 2], acc[i][j][half * 2 + 1], weight, gating));
                 }
+            } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const int n = n0 + wn * 32 + j * 8 + 2 * t + e;
+                        if (n >= N) continue;
+                        float v = acc[i][j][half * 2 + e];
+                        if (EPI == EXP_SQUARED_RELU) {
+                            v = fmaxf(v, 0.0f);
+                            v *= v;
+                        }
+                        Elem<O>::store(out + (int64_t)a * out_stride + n, v);
+                    }
+            }
         }
 }
 
 // ----------------------------------------------------------------------------- the weighted sum
 
 __global__ void expert_combine_kernel(const float* __restrict__ y, const float* __restrict__ weights,
-                                      const float* __restrict__ base, float* __restrict__ out, int width, int top) {
+                                      const float* __restrict__ base, const float* __restrict__ base_gate,
+                                      int64_t gate_stride, float* __restrict__ out, int width, int top) {
     pdl_trigger();
     pdl_wait();
     const int64_t row = blockIdx.x;
-    const float* w = weights + row * top;
+    const float* w = weights == nullptr ? nullptr : weights + row * top;
+    const float keep = base_gate == nullptr ? 1.0f : 1.0f / (1.0f + expf(-base_gate[row * gate_stride]));
     for (int j = blockIdx.y * blockDim.x + threadIdx.x; j < width; j += gridDim.y * blockDim.x) {
         float sum = 0.0f;
-        for (int s = 0; s < top; ++s) sum = fmaf(w[s], y[(row * top + s) * width + j], sum);
-        if (base != nullptr) sum += base[row * width + j];
+        for (int s = 0; s < top; ++s) sum = fmaf(w == nullptr ? 1.0f : w[s], y[(row * top + s) * width + j], sum);
+        if (base != nullptr) sum = fmaf(base[row * width + j], keep, sum);
         out[row * width + j] = sum;
     }
 }
 
 template <typename T, typename O>
 int launch_linear(const void* in, int64_t in_stride, const void* W, void* out, int64_t out_stride, const int* offsets,
-                  const int* order, int assignments, int experts, int top_div, int N, int K, int epilogue,
+                  const int* order, int assignments, int experts, int top_div, int N, int K, int epilogue, Gating gating,
                   cudaStream_t stream) {
     const dim3 grid((N + BN - 1) / BN, (assignments + BM - 1) / BM + experts);
     if (grid.y > 65535) return TB_ERR_BAD_SIZE;
-    cudaError_t launched;
-    if (epilogue == EXP_SQUARED_RELU)
-        launched = tb_launch_pdl(expert_linear_kernel<T, O, EXP_SQUARED_RELU>, grid, dim3(256), 0, stream, (const T*)in,
-                                 in_stride, (const T*)W, (O*)out, out_stride, offsets, order, experts, top_div, N, K);
-    else
-        launched = tb_launch_pdl(expert_linear_kernel<T, O, EXP_PLAIN>, grid, dim3(256), 0, stream, (const T*)in,
-                                 in_stride, (const T*)W, (O*)out, out_stride, offsets, order, experts, top_div, N, K);
-    return launched == cudaSuccess ? tb_launch_status() : (int)launched;
-}
-
-template <typename O, int EPI>
-int launch_linear_pipe(const void* in, int64_t in_stride, const void* W, void* out, int64_t out_stride,
-                       const int* offsets, const int* order, int assignments, int experts, int top_div, int N, int K,
-                       cudaStream_t stream) {
-    const dim3 grid((N + PN - 1) / PN, (assignments + PM - 1) / PM + experts);
-    if (grid.y > 65535) return TB_ERR_BAD_SIZE;
-    auto kernel = expert_linear_pipe_kernel<O, EPI>;
-    cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kPipeSmem);
-    if (err != cudaSuccess) return (int)err;
-    cudaError_t launched = tb_launch_pdl(kernel, grid, dim3(256), (size_t)kPipeSmem, stream, (const __nv_bfloat16*)in,
-                                         in_stride, (const __nv_bfloat16*)W, (O*)out, out_stride, offsets, order,
-                                         experts, top_div, N, K);
+    auto kernel = epilogue == EXP_GATED_CLAMPED  ? expert_linear_kernel<T, O, EXP_GATED_CLAMPED>
+                  : epilogue == EXP_SQUARED_RELU ? expert_linear_kernel<T, O, EXP_SQUARED_RELU>
+                                                 : expert_linear_kernel<T, O, EXP_PLAIN>;
+    cudaError_t launched = tb_launch_pdl(kernel, grid, dim3(256), 0, stream, (const T*)in, in_stride, (const T*)W, (O*)out,
+                                         out_stride, offsets, order, experts, top_div, N, K, gating);
     return launched == cudaSuccess ? tb_launch_status() : (int)launched;
 }
 
 template <typename O>
 int launch_linear_mma(const void* in, int64_t in_stride, const void* W, void* out, int64_t out_stride,
                       const int* offsets, const int* order, int assignments, int experts, int top_div, int N, int K,
-                      int epilogue, cudaStream_t stream) {
-    if (K % PK == 0)
-        return epilogue == EXP_SQUARED_RELU
-                   ? launch_linear_pipe<O, EXP_SQUARED_RELU>(in, in_stride, W, out, out_stride, offsets, order, assignments,
-                                                             experts, top_div, N, K, stream)
-                   : launch_linear_pipe<O, EXP_PLAIN>(in, in_stride, W, out, out_stride, offsets, order, assignments,
-                                                      experts, top_div, N, K, stream);
-    const dim3 grid((N + BN - 1) / BN, (assignments + BM - 1) / BM + experts);
+                      int epilogue, Gating gating, cudaStream_t stream) {
+    const bool pipe = K % PK == 0;
+    const int bm = pipe ? PM : BM, bn = pipe ? PN : BN;
+    const dim3 grid((N + bn - 1) / bn, (assignments + bm - 1) / bm + experts);
     if (grid.y > 65535) return TB_ERR_BAD_SIZE;
     cudaError_t launched;
-    if (epilogue == EXP_SQUARED_RELU)
-        launched = tb_launch_pdl(expert_linear_mma_kernel<O, EXP_SQUARED_RELU>, grid, dim3(128), 0, stream,
-                                 (const __nv_bfloat16*)in, in_stride, (const __nv_bfloat16*)W, (O*)out, out_stride,
-                                 offsets, order, experts, top_div, N, K);
-    else
-        launched = tb_launch_pdl(expert_linear_mma_kernel<O, EXP_PLAIN>, grid, dim3(128), 0, stream,
-                                 (const __nv_bfloat16*)in, in_stride, (const __nv_bfloat16*)W, (O*)out, out_stride,
-                                 offsets, order, experts, top_div, N, K);
+    if (pipe) {
+        auto kernel = epilogue == EXP_GATED_CLAMPED  ? expert_linear_pipe_kernel<O, EXP_GATED_CLAMPED>
+                      : epilogue == EXP_SQUARED_RELU ? expert_linear_pipe_kernel<O, EXP_SQUARED_RELU>
+                                                     : expert_linear_pipe_kernel<O, EXP_PLAIN>;
+        cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kPipeSmem);
+        if (err != cudaSuccess) return (int)err;
+        launched = tb_launch_pdl(kernel, grid, dim3(256), (size_t)kPipeSmem, stream, (const __nv_bfloat16*)in, in_stride,
+                                 (const __nv_bfloat16*)W, (O*)out, out_stride, offsets, order, experts, top_div, N, K, gating);
+    } else {
+        auto kernel = epilogue == EXP_GATED_CLAMPED  ? expert_linear_mma_kernel<O, EXP_GATED_CLAMPED>
+                      : epilogue == EXP_SQUARED_RELU ? expert_linear_mma_kernel<O, EXP_SQUARED_RELU>
+                                                     : expert_linear_mma_kernel<O, EXP_PLAIN>;
+        launched = tb_launch_pdl(kernel, grid, dim3(128), 0, stream, (const __nv_bfloat16*)in, in_stride,
+                                 (const __nv_bfloat16*)W, (O*)out, out_stride, offsets, order, experts, top_div, N, K, gating);
+    }
     return launched == cudaSuccess ? tb_launch_status() : (int)launched;
 }
 
@@ -612,6 +688,18 @@ TB_EXPORT int tb_choose_grouped(const float* logits, int* ids, float* weights, i
     return launched == cudaSuccess ? tb_launch_status() : (int)launched;
 }
 
+// logits: 32-bit, row stride `stride` >= experts; the first `experts` numbers of a row are the router's.
+TB_EXPORT int tb_choose_sigmoid(const float* logits, int64_t stride, int* ids, float* weights, int rows, int experts, int top,
+                                cudaStream_t stream) {
+    if (rows == 0) return 0;
+    if (experts < 1 || top < 1 || top > experts || stride < experts) return TB_ERR_BAD_SIZE;
+    const size_t smem = (size_t)kRouteWarps * experts * sizeof(float);
+    if (smem > 40 * 1024) return TB_ERR_BAD_SIZE;
+    cudaError_t launched = tb_launch_pdl(choose_sigmoid_kernel, dim3((rows + kRouteWarps - 1) / kRouteWarps),
+                                         dim3(kRouteWarps * 32), smem, stream, logits, stride, ids, weights, rows, experts, top);
+    return launched == cudaSuccess ? tb_launch_status() : (int)launched;
+}
+
 // ids: int32 [assignments]; offsets: int32 [experts + 1]; order: int32 [assignments].
 TB_EXPORT int tb_expert_plan(const int* ids, int assignments, int experts, int* offsets, int* order,
                              cudaStream_t stream) {
@@ -622,47 +710,51 @@ TB_EXPORT int tb_expert_plan(const int* ids, int assignments, int experts, int* 
 }
 
 // in: [*, K] of dtype (row stride in_stride); W: [experts, N, K] of dtype; out: [assignments, N] of out_dtype (row
-// stride out_stride); top_div: the source row of assignment a is a / top_div.  epilogue: 0 plain, 1 squared ReLU.
+// stride out_stride); top_div: the source row of assignment a is a / top_div.  epilogue: 0 plain, 1 squared ReLU, 2 gated
+// (N even, gate and up rows alternating, out [assignments, N / 2]; row_weights: null or 32-bit [assignments]).
 // tensor_cores != 0 asks for the mma.sync kernels (bfloat16, K a multiple of 32, 16-byte aligned rows; the pipelined
 // one where K is a multiple of 64); the entry point refuses it where it cannot run.
 TB_EXPORT int tb_expert_linear(const void* in, int64_t in_stride, const void* W, void* out, int64_t out_stride,
                                const int* offsets, const int* order, int assignments, int experts, int top_div, int N,
-                               int K, int epilogue, int dtype, int out_dtype, int tensor_cores, cudaStream_t stream) {
+                               int K, int epilogue, const float* row_weights, float limit, float slope, int dtype,
+                               int out_dtype, int tensor_cores, cudaStream_t stream) {
     if (assignments == 0 || N == 0) return 0;
     if (K < 1 || top_div < 1 || experts < 1) return TB_ERR_BAD_SIZE;
-    if (epilogue != EXP_PLAIN && epilogue != EXP_SQUARED_RELU) return TB_ERR_BAD_SIZE;
+    if (epilogue < EXP_PLAIN || epilogue > EXP_GATED_CLAMPED || (epilogue == EXP_GATED_CLAMPED && N % 2 != 0)) return TB_ERR_BAD_SIZE;
+    Gating gating;
+    gating.row_weights = row_weights; gating.limit = limit; gating.slope = slope;
     if (tensor_cores) {
         if (dtype != TB_BF16) return TB_ERR_BAD_DTYPE;
         if (K % MK != 0 || in_stride % 8 != 0 || ((uintptr_t)in | (uintptr_t)W) % 16 != 0) return TB_ERR_BAD_ALIGN;
         if (out_dtype == TB_F32)
             return launch_linear_mma<float>(in, in_stride, W, out, out_stride, offsets, order, assignments, experts,
-                                            top_div, N, K, epilogue, stream);
+                                            top_div, N, K, epilogue, gating, stream);
         if (out_dtype == TB_BF16)
             return launch_linear_mma<__nv_bfloat16>(in, in_stride, W, out, out_stride, offsets, order, assignments,
-                                                    experts, top_div, N, K, epilogue, stream);
+                                                    experts, top_div, N, K, epilogue, gating, stream);
         return TB_ERR_BAD_DTYPE;
     }
     if (dtype == TB_F32 && out_dtype == TB_F32)
         return launch_linear<float, float>(in, in_stride, W, out, out_stride, offsets, order, assignments, experts,
-                                           top_div, N, K, epilogue, stream);
+                                           top_div, N, K, epilogue, gating, stream);
     if (dtype == TB_BF16 && out_dtype == TB_F32)
         return launch_linear<__nv_bfloat16, float>(in, in_stride, W, out, out_stride, offsets, order, assignments,
-                                                   experts, top_div, N, K, epilogue, stream);
+                                                   experts, top_div, N, K, epilogue, gating, stream);
     if (dtype == TB_BF16 && out_dtype == TB_BF16)
         return launch_linear<__nv_bfloat16, __nv_bfloat16>(in, in_stride, W, out, out_stride, offsets, order,
-                                                           assignments, experts, top_div, N, K, epilogue, stream);
+                                                           assignments, experts, top_div, N, K, epilogue, gating, stream);
     return TB_ERR_BAD_DTYPE;
 }
 
-// y: 32-bit [rows * top, width]; weights: 32-bit [rows, top]; base: null or 32-bit [rows, width]; out: 32-bit
-// [rows, width] (may alias base).
-TB_EXPORT int tb_expert_combine(const float* y, const float* weights, const float* base, float* out, int rows,
-                                int width, int top, cudaStream_t stream) {
+// y: 32-bit [rows * top, width]; weights: null or 32-bit [rows, top]; base: null or 32-bit [rows, width]; base_gate: null
+// or a 32-bit number per row (stride gate_stride); out: 32-bit [rows, width] (may alias base).
+TB_EXPORT int tb_expert_combine(const float* y, const float* weights, const float* base, const float* base_gate,
+                                int64_t gate_stride, float* out, int rows, int width, int top, cudaStream_t stream) {
     if (rows == 0 || width == 0) return 0;
     if (top < 1) return TB_ERR_BAD_SIZE;
     int by = (width + 255) / 256;
     if (by > 32) by = 32;
     cudaError_t launched = tb_launch_pdl(expert_combine_kernel, dim3(rows, by), dim3(256), 0, stream, y, weights, base,
-                                         out, width, top);
+                                         base_gate, gate_stride, out, width, top);
     return launched == cudaSuccess ? tb_launch_status() : (int)launched;
 }

@@ -4,7 +4,8 @@
 //   tb_gated_activation   out[t, j] = act(gate[t, j] + bg[j]) * (up[t, j] + bu[j]); gate and up are the two halves
 //                         of a row of `gu`; the biases (32-bit, [2 * inter], gate then up) may be null.
 //                         act: 0 = SiLU, 1 = GELU in its tanh form
-//                         0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
+//                         0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))); 2 = both halves clamped: with
+//                         g = min(gate, limit) and u = min(max(up, -limit), limit), g * sigmoid(slope * g) * (u + 1).
 //   tb_squared_relu       out[t, j] = max(z[t, j], 0)^2
 //   tb_add_bias           y[t, j] += b[j]                      (y 32-bit or bfloat16, b 32-bit)
 //   tb_scale_rows         y[t, j] *= s                         (32-bit y)
@@ -18,7 +19,7 @@
 
 namespace {
 
-enum Activation : int { ACT_SILU = 0, ACT_GELU_TANH = 1 };
+enum Activation : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_CLAMPED = 2 };
 
 template <int ACT>
 __device__ __forceinline__ float activate(float z) {
@@ -27,9 +28,17 @@ __device__ __forceinline__ float activate(float z) {
     return 0.5f * z * (1.0f + tanhf(inner));
 }
 
+template <int ACT>
+__device__ __forceinline__ float gated(float g, float u, float limit, float slope) {
+    if (ACT != ACT_CLAMPED) return activate<ACT>(g) * u;
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * (1.0f / (1.0f + expf(-slope * g))) * (u + 1.0f);
+}
+
 template <typename T, int ACT>
 __global__ void gated_activation_kernel(const T* __restrict__ gu, int64_t gu_stride, const float* __restrict__ bias,
-                                        T* __restrict__ out, int64_t out_stride, int inter) {
+                                        T* __restrict__ out, int64_t out_stride, int inter, float limit, float slope) {
     pdl_trigger();
     pdl_wait();
     const T* g = gu + (int64_t)blockIdx.x * gu_stride;
@@ -40,7 +49,7 @@ __global__ void gated_activation_kernel(const T* __restrict__ gu, int64_t gu_str
             gv += bias[j];
             uv += bias[inter + j];
         }
-        Elem<T>::store(o + j, activate<ACT>(gv) * uv);
+        Elem<T>::store(o + j, gated<ACT>(gv, uv, limit, slope));
     }
 }
 
@@ -48,7 +57,7 @@ __global__ void gated_activation_kernel(const T* __restrict__ gu, int64_t gu_str
 template <typename T, int ACT>
 __global__ void gated_activation_packets_kernel(const T* __restrict__ gu, int64_t gu_stride,
                                                 const float* __restrict__ bias, T* __restrict__ out,
-                                                int64_t out_stride, int inter) {
+                                                int64_t out_stride, int inter, float limit, float slope) {
     constexpr int N = Packet<T>::N;
     pdl_trigger();
     pdl_wait();
@@ -64,7 +73,7 @@ __global__ void gated_activation_packets_kernel(const T* __restrict__ gu, int64_
                 gv[e] += bias[j + e];
                 uv[e] += bias[inter + j + e];
             }
-            ov[e] = activate<ACT>(gv[e]) * uv[e];
+            ov[e] = gated<ACT>(gv[e], uv[e], limit, slope);
         }
         Packet<T>::store(o + j, ov);
     }
@@ -185,7 +194,7 @@ inline int grid_for(int64_t total, int threads) {
 
 template <typename T, int ACT>
 int launch_gated(const void* gu, int64_t gu_stride, const float* bias, void* out, int64_t out_stride, int rows, int inter,
-                 cudaStream_t stream) {
+                 float limit, float slope, cudaStream_t stream) {
     constexpr int N = Packet<T>::N;
     const int threads = 256;
     const bool packets = inter % N == 0 && gu_stride % N == 0 && out_stride % N == 0 &&
@@ -193,28 +202,30 @@ int launch_gated(const void* gu, int64_t gu_stride, const float* bias, void* out
     cudaError_t launched;
     if (packets)
         launched = tb_launch_pdl(gated_activation_packets_kernel<T, ACT>, row_grid(rows, inter, threads, N), dim3(threads),
-                                 0, stream, (const T*)gu, gu_stride, bias, (T*)out, out_stride, inter);
+                                 0, stream, (const T*)gu, gu_stride, bias, (T*)out, out_stride, inter, limit, slope);
     else
         launched = tb_launch_pdl(gated_activation_kernel<T, ACT>, row_grid(rows, inter, threads), dim3(threads), 0,
-                                 stream, (const T*)gu, gu_stride, bias, (T*)out, out_stride, inter);
+                                 stream, (const T*)gu, gu_stride, bias, (T*)out, out_stride, inter, limit, slope);
     return launched == cudaSuccess ? tb_launch_status() : (int)launched;
 }
 
 }  // namespace
 
+// limit, slope: only activation 2 reads them.
 TB_EXPORT int tb_gated_activation(const void* gu, int64_t gu_stride, const float* bias, void* out, int64_t out_stride,
-                                  int rows, int inter, int activation, int dtype, cudaStream_t stream) {
+                                  int rows, int inter, int activation, float limit, float slope, int dtype,
+                                  cudaStream_t stream) {
     if (rows == 0 || inter == 0) return 0;
-    if (activation != ACT_SILU && activation != ACT_GELU_TANH) return TB_ERR_BAD_SIZE;
-    if (dtype == TB_F32)
-        return activation == ACT_SILU
-                   ? launch_gated<float, ACT_SILU>(gu, gu_stride, bias, out, out_stride, rows, inter, stream)
-                   : launch_gated<float, ACT_GELU_TANH>(gu, gu_stride, bias, out, out_stride, rows, inter, stream);
-    if (dtype == TB_BF16)
-        return activation == ACT_SILU
-                   ? launch_gated<__nv_bfloat16, ACT_SILU>(gu, gu_stride, bias, out, out_stride, rows, inter, stream)
-                   : launch_gated<__nv_bfloat16, ACT_GELU_TANH>(gu, gu_stride, bias, out, out_stride, rows, inter, stream);
-    return TB_ERR_BAD_DTYPE;
+    if (activation < ACT_SILU || activation > ACT_CLAMPED) return TB_ERR_BAD_SIZE;
+    if (dtype != TB_F32 && dtype != TB_BF16) return TB_ERR_BAD_DTYPE;
+#define TB_RUN(ACT)                                                                                                   \
+    return dtype == TB_F32                                                                                            \
+               ? launch_gated<float, ACT>(gu, gu_stride, bias, out, out_stride, rows, inter, limit, slope, stream)    \
+               : launch_gated<__nv_bfloat16, ACT>(gu, gu_stride, bias, out, out_stride, rows, inter, limit, slope, stream)
+    if (activation == ACT_SILU) TB_RUN(ACT_SILU);
+    if (activation == ACT_GELU_TANH) TB_RUN(ACT_GELU_TANH);
+    TB_RUN(ACT_CLAMPED);
+#undef TB_RUN
 }
 
 TB_EXPORT int tb_squared_relu(const void* z, int64_t z_stride, void* out, int64_t out_stride, int rows, int width,

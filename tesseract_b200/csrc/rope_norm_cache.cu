@@ -9,7 +9,12 @@
 // sqrt(mean(head^2) + eps), the mean over all d numbers of the rotated head.  Queries go to q_out, keys and values
 // into the pages: a page is [G][page_size][d] keys followed by [G][page_size][dv] values.
 //
-// One warp per (row, head of q, k or v).  All arithmetic is 32-bit; each stored value is rounded once; the order
+// Values may also be mixed with those of an earlier layer: `value_mode` 1 leaves this layer's values (bias added, 32-bit,
+// [rows, G * dv]) in `first_values` for later layers, 2 stores (1 - mix) * v + mix * first_values instead of v, `mix` one
+// number on the device.
+//
+// One warp per (row, head of q, k or v); rows that neither turn nor are normed take a kernel of their own, a thread a
+// 16-byte packet of the row.  All arithmetic is 32-bit; each stored value is rounded once; the order
 // of a head's sum of squares depends on d alone.
 //
 // tb_pool_blocks, for a mixer that also attends to averaged blocks of old tokens, runs behind it: every row that ends a
@@ -28,12 +33,19 @@ struct HeadGeometry {
     float amplitude, eps;
 };
 
+enum ValueMode : int { VALUES_PLAIN = 0, VALUES_LEAVE = 1, VALUES_MIX = 2 };
+struct ValueMix {
+    int mode;
+    float* first;                        // [rows, G * dv]
+    const float* mix;                    // one number
+};
+
 template <typename T>
 __global__ void __launch_bounds__(kWarps * 32)
 rope_norm_cache_kernel(const T* __restrict__ proj, int64_t proj_stride, T* __restrict__ q_out, int64_t q_stride,
                        T* __restrict__ cache, const int* __restrict__ positions, const int* __restrict__ seq_of_row,
                        const int* __restrict__ block_table, int bt_stride, const float* __restrict__ inv_freq,
-                       const float* __restrict__ bias, HeadGeometry g, int write_kv) {
+                       const float* __restrict__ bias, HeadGeometry g, int write_kv, ValueMix values) {
     extern __shared__ float head_cache[];             // kWarps * dim
     pdl_trigger();
     pdl_wait();                                       // the projected rows and the step's metadata come from kernels in front
@@ -61,7 +73,16 @@ rope_norm_cache_kernel(const T* __restrict__ proj, int64_t proj_stride, T* __res
             dst += (int64_t)g.kv_heads * g.page_size * g.dim + ((int64_t)head * g.page_size + in_page) * g.vdim;
             const int64_t at = (int64_t)(g.heads + g.kv_heads) * g.dim + (int64_t)head * g.vdim;
             const T* src = prow + at;
-            if (bias == nullptr) {
+            if (values.mode != VALUES_PLAIN) {
+                float* first = values.first + (int64_t)row * g.kv_heads * g.vdim + (int64_t)head * g.vdim;
+                const float mix = values.mode == VALUES_MIX ? *values.mix : 0.0f;
+                for (int i = lane; i < g.vdim; i += 32) {
+                    float v = Elem<T>::load(src + i) + (bias != nullptr ? bias[at + i] : 0.0f);
+                    if (values.mode == VALUES_LEAVE) first[i] = v;
+                    else v = fmaf(mix, first[i], (1.0f - mix) * v);
+                    Elem<T>::store(dst + i, v);
+                }
+            } else if (bias == nullptr) {
                 for (int i = lane; i < g.vdim; i += 32) dst[i] = src[i];
             } else {
                 for (int i = lane; i < g.vdim; i += 32) Elem<T>::store(dst + i, Elem<T>::load(src + i) + bias[at + i]);
@@ -104,6 +125,94 @@ rope_norm_cache_kernel(const T* __restrict__ proj, int64_t proj_stride, T* __res
     for (int i = lane; i < g.dim; i += 32) Elem<T>::store(dst + i, mine[i] * inv);
 }
 
+
+// Rows that neither turn nor are normed: a thread a 16-byte packet of a row's q, k and v (head sizes that are multiples of a
+// packet, aligned rows).
+template <typename T>
+__global__ void __launch_bounds__(128)
+bias_cache_packets_kernel(const T* __restrict__ proj, int64_t proj_stride, T* __restrict__ q_out, int64_t q_stride,
+                          T* __restrict__ cache, const int* __restrict__ positions, const int* __restrict__ seq_of_row,
+                          const int* __restrict__ block_table, int bt_stride, const float* __restrict__ bias, HeadGeometry g,
+                          int write_kv, ValueMix values) {
+    constexpr int N = Packet<T>::N;
+    const int row = blockIdx.x;
+    const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * N;
+    const int q_width = g.heads * g.dim, k_end = q_width + g.kv_heads * g.dim, end = k_end + g.kv_heads * g.vdim;
+    pdl_trigger();
+    pdl_wait();
+    if (c0 >= end) return;
+    float v[N];
+    Packet<T>::load(proj + (int64_t)row * proj_stride + c0, v);
+    if (bias != nullptr) {
+#pragma unroll
+        for (int e = 0; e < N; e += 4) {
+            const float4 b = *reinterpret_cast<const float4*>(bias + c0 + e);
+            v[e] += b.x; v[e + 1] += b.y; v[e + 2] += b.z; v[e + 3] += b.w;
+        }
+    }
+    if (c0 < q_width) {
+        Packet<T>::store(q_out + (int64_t)row * q_stride + c0, v);
+        return;
+    }
+    const bool is_value = c0 >= k_end;
+    if (is_value && values.mode != VALUES_PLAIN) {
+        float* first = values.first + (int64_t)row * g.kv_heads * g.vdim + (c0 - k_end);
+        if (values.mode == VALUES_LEAVE) {
+#pragma unroll
+            for (int e = 0; e < N; e += 4) *reinterpret_cast<float4*>(first + e) = make_float4(v[e], v[e + 1], v[e + 2], v[e + 3]);
+        } else {
+            const float mix = *values.mix;
+#pragma unroll
+            for (int e = 0; e < N; e += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(first + e);
+                v[e] = fmaf(mix, f.x, (1.0f - mix) * v[e]);
+                v[e + 1] = fmaf(mix, f.y, (1.0f - mix) * v[e + 1]);
+                v[e + 2] = fmaf(mix, f.z, (1.0f - mix) * v[e + 2]);
+                v[e + 3] = fmaf(mix, f.w, (1.0f - mix) * v[e + 3]);
+            }
+        }
+    }
+    if (!write_kv) return;
+    const int pos = positions[row];
+    const int page = block_table[(int64_t)seq_of_row[row] * bt_stride + pos / g.page_size], in_page = pos % g.page_size;
+    T* dst = cache + (int64_t)page * g.kv_heads * g.page_size * (g.dim + g.vdim);
+    if (is_value) {
+        const int head = (c0 - k_end) / g.vdim, e0 = (c0 - k_end) % g.vdim;
+        dst += (int64_t)g.kv_heads * g.page_size * g.dim + ((int64_t)head * g.page_size + in_page) * g.vdim + e0;
+    } else {
+        const int head = (c0 - q_width) / g.dim, e0 = (c0 - q_width) % g.dim;
+        dst += ((int64_t)head * g.page_size + in_page) * g.dim + e0;
+    }
+    Packet<T>::store(dst, v);
+}
+
+template <typename T>
+int launch_rope_norm(const void* proj, int64_t proj_stride, void* q_out, int64_t q_stride, void* cache, const int* positions,
+                     const int* seq_of_row, const int* block_table, int bt_stride, const float* inv_freq, const float* bias,
+                     int rows, const HeadGeometry& g, int write_kv, const ValueMix& values, cudaStream_t stream) {
+    constexpr int N = Packet<T>::N;
+    const uintptr_t bits = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache | (uintptr_t)bias | (uintptr_t)values.first;
+    cudaError_t launched;
+    if (g.rot_dims == 0 && !g.unit_norm && g.dim % N == 0 && g.vdim % N == 0 && proj_stride % N == 0 && q_stride % N == 0 &&
+        bits % 16 == 0) {
+        const int packets = (g.heads * g.dim + g.kv_heads * (g.dim + g.vdim)) / N;
+        const dim3 grid(rows, (packets + 127) / 128);
+        if (grid.y > 65535) return TB_ERR_BAD_SIZE;
+        launched = tb_launch_pdl(bias_cache_packets_kernel<T>, grid, dim3(128), 0, stream, (const T*)proj, proj_stride,
+                                 (T*)q_out, q_stride, (T*)cache, positions, seq_of_row, block_table, bt_stride, bias, g,
+                                 write_kv, values);
+    } else {
+        const size_t smem = (size_t)kWarps * g.dim * sizeof(float);
+        if (smem > 40 * 1024) return TB_ERR_BAD_SIZE;
+        const int slots = g.heads + 2 * g.kv_heads;
+        const dim3 grid(rows, (slots + kWarps - 1) / kWarps);
+        if (grid.y > 65535) return TB_ERR_BAD_SIZE;
+        launched = tb_launch_pdl(rope_norm_cache_kernel<T>, grid, dim3(kWarps * 32), smem, stream, (const T*)proj, proj_stride,
+                                 (T*)q_out, q_stride, (T*)cache, positions, seq_of_row, block_table, bt_stride, inv_freq,
+                                 bias, g, write_kv, values);
+    }
+    return launched == cudaSuccess ? tb_launch_status() : (int)launched;
+}
 
 // For every row of the step that ends a block of `pool` positions ((position + 1) % pool == 0): the averages of the block's
 // keys and of its values, as the pages hold them, into entry position / pool of the request's pooled pages (same page
@@ -150,37 +259,33 @@ pool_blocks_kernel(const T* __restrict__ cache, T* __restrict__ pool_cache, cons
 
 // proj: [rows, >= (H + G) * d + G * dv] with row stride proj_stride (elements); q_out: [rows, H * d] with row
 // stride q_stride; cache: this layer's pages; inv_freq: 32-bit [rot_dims / 2] (may be null when rot_dims is 0); bias:
-// null or 32-bit [(H + G) * d + G * dv].
+// null or 32-bit [(H + G) * d + G * dv].  value_mode: 0 values as they are, 1 also left in first_values (32-bit [rows, G * dv]),
+// 2 mixed with first_values by *value_mix.
 TB_EXPORT int tb_rope_norm_cache(const void* proj, int64_t proj_stride, void* q_out, int64_t q_stride, void* cache,
                                  const int* positions, const int* seq_of_row, const int* block_table, int bt_stride,
                                  const float* inv_freq, const float* bias, float amplitude, int rows, int heads, int kv_heads, int dim,
                                  int vdim, int rot_dims, int unit_norm, float eps, int page_size, int write_kv,
-                                 int dtype, cudaStream_t stream) {
+                                 int value_mode, float* first_values, const float* value_mix, int dtype,
+                                 cudaStream_t stream) {
     if (rows == 0) return 0;
+    if (value_mode < VALUES_PLAIN || value_mode > VALUES_MIX || (value_mode != VALUES_PLAIN && first_values == nullptr) ||
+        (value_mode == VALUES_MIX && value_mix == nullptr))
+        return TB_ERR_BAD_SIZE;
     if (heads < 1 || kv_heads < 1 || dim < 1 || vdim < 1 || page_size < 1) return TB_ERR_BAD_SIZE;
     if (rot_dims < 0 || rot_dims > dim || rot_dims % 2 != 0) return TB_ERR_BAD_SIZE;
     if (rot_dims > 0 && inv_freq == nullptr) return TB_ERR_BAD_SIZE;
-    const size_t smem = (size_t)kWarps * dim * sizeof(float);
-    if (smem > 40 * 1024) return TB_ERR_BAD_SIZE;
     HeadGeometry g;
     g.heads = heads; g.kv_heads = kv_heads; g.dim = dim; g.vdim = vdim; g.rot_dims = rot_dims; g.page_size = page_size;
     g.unit_norm = unit_norm; g.amplitude = amplitude; g.eps = eps;
-    const int slots = heads + 2 * kv_heads;
-    const dim3 grid(rows, (slots + kWarps - 1) / kWarps);
-    if (grid.y > 65535) return TB_ERR_BAD_SIZE;
-    cudaError_t launched;
+    ValueMix values;
+    values.mode = value_mode; values.first = first_values; values.mix = value_mix;
     if (dtype == TB_F32)
-        launched = tb_launch_pdl(rope_norm_cache_kernel<float>, grid, dim3(kWarps * 32), smem, stream, (const float*)proj,
-                                 proj_stride, (float*)q_out, q_stride, (float*)cache, positions, seq_of_row, block_table,
-                                 bt_stride, inv_freq, bias, g, write_kv);
-    else if (dtype == TB_BF16)
-        launched = tb_launch_pdl(rope_norm_cache_kernel<__nv_bfloat16>, grid, dim3(kWarps * 32), smem, stream,
-                                 (const __nv_bfloat16*)proj, proj_stride, (__nv_bfloat16*)q_out, q_stride,
-                                 (__nv_bfloat16*)cache, positions, seq_of_row, block_table, bt_stride, inv_freq, bias, g,
-                                 write_kv);
-    else
-        return TB_ERR_BAD_DTYPE;
-    return launched == cudaSuccess ? tb_launch_status() : (int)launched;
+        return launch_rope_norm<float>(proj, proj_stride, q_out, q_stride, cache, positions, seq_of_row, block_table,
+                                       bt_stride, inv_freq, bias, rows, g, write_kv, values, stream);
+    if (dtype == TB_BF16)
+        return launch_rope_norm<__nv_bfloat16>(proj, proj_stride, q_out, q_stride, cache, positions, seq_of_row, block_table,
+                                               bt_stride, inv_freq, bias, rows, g, write_kv, values, stream);
+    return TB_ERR_BAD_DTYPE;
 }
 
 // cache: the layer's pages of keys and values ([G][page_size][d] keys then [G][page_size][dv] values a page), already

@@ -813,7 +813,7 @@ def attention_masked(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
                      positions: torch.Tensor, seq_of_row: torch.Tensor, block_table: torch.Tensor, *, heads: int,
                      kv_heads: int, dim: int, vdim: int, page_size: int, mask_kind: int, mask_size: int, sink: bool,
                      scale: float, keys_per_value: int = 1, sinks: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                     pooled=None) -> torch.Tensor:
+                     pooled=None, keep_first: int = 0, distance_bias=None) -> torch.Tensor:
     """Paged attention with 32-bit scores and weights: ``q`` ``[T, heads * dim]``, optional ``gate``
     ``[T, heads * vdim]`` (the output is multiplied by its sigmoid), ``out`` ``[T, heads * vdim]`` in the dtype of ``q``
     or in float32 (the weighted sums as they are, unrounded); pages hold ``[kv_heads, page_size, dim]`` keys then
@@ -823,7 +823,9 @@ def attention_masked(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
     averaged key and value per block of ``pool`` positions that ends in front of the window, from
     ``pooled = (pages of the averages, their block table, pool)``; ``sink``: one more entry of score 0 in the softmax's
     denominator, or, with ``sinks`` (float32 ``[heads]``), of a learned score per head; ``softcap`` > 0: a score ``s``
-    becomes ``softcap * tanh(s / softcap)``."""
+    becomes ``softcap * tanh(s / softcap)``; ``keep_first`` (with ``MASK_WINDOW``): the first positions of the sequence that
+    every row sees although its window has passed them; ``distance_bias = (weight, rate)`` (float32 ``[heads]`` each): the
+    score of the key ``n`` positions back loses ``weight * ln(1 + rate * n)``."""
     _cuda(q, gate, out, cache, positions, seq_of_row, block_table)
     rows = q.shape[0]
     _need(q.stride(1) == 1 and q.shape[1] == heads * dim, "attention_masked q")
@@ -834,7 +836,7 @@ def attention_masked(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
     _need(cache.dtype == q.dtype and cache.is_contiguous(), "attention_masked cache")
     if gate is not None:
         _need(gate.stride(1) == 1 and gate.shape == (rows, heads * vdim) and gate.dtype == q.dtype, "attention_masked gate")
-    extras = _mask_extras("attention_masked", q, heads, mask_kind, keys_per_value, sinks, pooled)
+    extras = _mask_extras("attention_masked", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias)
     lib = load_library("attention_masked")
     _check(lib.tb_attention_masked(_ptr(q), _i64(q.stride(0)), _ptr(gate), _i64(gate.stride(0) if gate is not None else 0),
                                    _ptr(out), _i64(out.stride(0)), _ptr(cache), _ptr(positions), _ptr(seq_of_row),
@@ -846,8 +848,17 @@ def attention_masked(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
     return out
 
 
-def _mask_extras(what: str, q: torch.Tensor, heads: int, mask_kind: int, keys_per_value: int, sinks, pooled):
-    """The arguments a learned sink and pooled blocks add to an attention kernel's call, checked."""
+def _mask_extras(what: str, q: torch.Tensor, heads: int, mask_kind: int, keys_per_value: int, sinks, pooled, keep_first,
+                 distance_bias):
+    """The arguments that a learned sink, pooled blocks, kept first positions and a distance bias add to an attention
+    kernel's call, checked."""
+    weight = rate = None
+    if distance_bias is not None:
+        weight, rate = distance_bias
+        _cuda(weight, rate)
+        for v in (weight, rate):
+            _need(v.dtype == torch.float32 and v.numel() == heads and v.is_contiguous(), f"{what} distance bias")
+    _need(keep_first == 0 or (keep_first > 0 and mask_kind == MASK_WINDOW), f"{what}: only a window keeps first positions")
     if sinks is not None:
         _cuda(sinks)
         _need(sinks.dtype == torch.float32 and sinks.numel() == heads and sinks.is_contiguous(), f"{what} sinks")
@@ -859,7 +870,8 @@ def _mask_extras(what: str, q: torch.Tensor, heads: int, mask_kind: int, keys_pe
         _cuda(pool_cache, pool_table)
         _need(pool_cache.dtype == q.dtype and pool_cache.is_contiguous() and pool_table.dtype == torch.int32
               and pool_table.stride(1) == 1 and pool >= 1, f"{what} pooled pages")
-    return (_ptr(pool_cache), _ptr(pool_table), _i32(pool_table.stride(0) if pool_table is not None else 0), _i32(pool))
+    return (_ptr(pool_cache), _ptr(pool_table), _i32(pool_table.stride(0) if pool_table is not None else 0), _i32(pool),
+            _i32(keep_first), _ptr(weight), _ptr(rate))
 
 
 def attention_prompt_mma_supported(dtype: torch.dtype, dim: int, vdim: int) -> bool:
@@ -872,7 +884,7 @@ def attention_prompt_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor
                          row_start: torch.Tensor, block_table: torch.Tensor, *, num_seqs: int, heads: int,
                          kv_heads: int, dim: int, vdim: int, page_size: int, mask_kind: int, mask_size: int,
                          scale: float, keys_per_value: int = 1, sinks: Optional[torch.Tensor] = None,
-                         softcap: float = 0.0, pooled=None) -> torch.Tensor:
+                         softcap: float = 0.0, pooled=None, keep_first: int = 0, distance_bias=None) -> torch.Tensor:
     """:func:`attention_masked` (no fixed sink, no gate; ``sinks``, ``softcap`` and ``pooled`` as there) for bfloat16 prompt portions on the tensor cores: scores from
     exact bfloat16 products with 32-bit accumulation, 32-bit softmax, the 32-bit weights split in two bfloat16 halves
     for the product with the values.  The rows of a sequence (``row_start``) stand at consecutive positions.  ``out`` in
@@ -885,7 +897,7 @@ def attention_prompt_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor
     _need(keys_per_value >= 1 and kv_heads % keys_per_value == 0, "attention_prompt_mma keys_per_value")
     _need(cache.dtype == q.dtype and cache.is_contiguous(), "attention_prompt_mma cache")
     _need(row_start.dtype == torch.int32 and row_start.numel() >= num_seqs + 1, "attention_prompt_mma row_start")
-    extras = _mask_extras("attention_prompt_mma", q, heads, mask_kind, keys_per_value, sinks, pooled)
+    extras = _mask_extras("attention_prompt_mma", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias)
     lib = load_library("attention_prompt_mma")
     _check(lib.tb_attention_prompt_mma(_ptr(q), _i64(q.stride(0)), _ptr(out), _i64(out.stride(0)), _ptr(cache),
                                        _ptr(positions), _ptr(row_start), _ptr(block_table), _i32(block_table.stride(0)),
@@ -901,7 +913,7 @@ def attention_rows_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
                        seq_of_row: torch.Tensor, block_table: torch.Tensor, *, heads: int, kv_heads: int, dim: int,
                        vdim: int, page_size: int, mask_kind: int, mask_size: int, scale: float,
                        keys_per_value: int = 1, sinks: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                       pooled=None) -> torch.Tensor:
+                       pooled=None, keep_first: int = 0, distance_bias=None) -> torch.Tensor:
     """:func:`attention_prompt_mma` for steps of few rows at any positions: a block a (row, kv head), the kv head's
     query heads (at most 16) side by side in the tensor-core tile."""
     _cuda(q, out, cache, positions, seq_of_row, block_table)
@@ -911,7 +923,7 @@ def attention_rows_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
           "attention_rows_mma out")
     _need(keys_per_value >= 1 and kv_heads % keys_per_value == 0, "attention_rows_mma keys_per_value")
     _need(cache.dtype == q.dtype and cache.is_contiguous(), "attention_rows_mma cache")
-    extras = _mask_extras("attention_rows_mma", q, heads, mask_kind, keys_per_value, sinks, pooled)
+    extras = _mask_extras("attention_rows_mma", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias)
     lib = load_library("attention_prompt_mma")
     _check(lib.tb_attention_rows_mma(_ptr(q), _i64(q.stride(0)), _ptr(out), _i64(out.stride(0)), _ptr(cache),
                                      _ptr(positions), _ptr(seq_of_row), _ptr(block_table), _i32(block_table.stride(0)),
@@ -940,6 +952,118 @@ def gated_recurrence(proj: torch.Tensor, bias_z: torch.Tensor, bias_x: torch.Ten
                                    _ptr(state_slots), _i32(num_seqs), _i32(width), _i32(max_new), _stream()),
            "gated_recurrence")
     return out
+
+
+def short_conv(proj: torch.Tensor, in_bias: Optional[torch.Tensor], taps: torch.Tensor, out_bias: Optional[torch.Tensor],
+               state: Optional[torch.Tensor], out: torch.Tensor, positions: torch.Tensor, seq_of_row: torch.Tensor,
+               row_start: torch.Tensor, seq_begin: torch.Tensor, state_slots: torch.Tensor, *, num_seqs: int,
+               single: bool) -> torch.Tensor:
+    """A causal convolution per channel of ``proj + in_bias`` (``[T, C]``; ``taps`` float32 ``[J, C]``, oldest first) plus
+    ``out_bias``; ``state`` (float32 ``[slots, J - 1, C]``; None for one tap) holds each request's last ``J - 1`` rows of
+    ``proj + in_bias`` and is renewed.  ``single``: every sequence brings one row (the state is renewed inside the kernel);
+    otherwise a second launch renews it."""
+    _cuda(proj, in_bias, taps, out_bias, state, out, positions, seq_of_row, row_start, seq_begin, state_slots)
+    rows, channels = out.shape
+    count = taps.shape[0]
+    _need(proj.stride(1) == 1 and tuple(proj.shape) == (rows, channels) and out.stride(1) == 1 and out.dtype == proj.dtype,
+          "short_conv proj/out")
+    _need(taps.dtype == torch.float32 and taps.is_contiguous() and taps.shape[1] == channels, "short_conv taps")
+    for b in (in_bias, out_bias):
+        _need(b is None or (b.dtype == torch.float32 and b.numel() == channels and b.is_contiguous()), "short_conv bias")
+    if count > 1:
+        _need(state is not None and state.dtype == torch.float32 and state.is_contiguous()
+              and tuple(state.shape[1:]) == (count - 1, channels), "short_conv state")
+    for t in (positions, seq_of_row, row_start, seq_begin, state_slots):
+        _need(t.dtype == torch.int32, "short_conv metadata must be int32")
+    lib = load_library("short_conv")
+    _check(lib.tb_short_conv(_ptr(proj), _i64(proj.stride(0)), _ptr(in_bias), _ptr(taps), _ptr(out_bias), _ptr(state), _ptr(out),
+                             _i64(out.stride(0)), _ptr(positions), _ptr(seq_of_row), _ptr(row_start), _ptr(seq_begin),
+                             _ptr(state_slots), _i32(rows), _i32(channels), _i32(count), _i32(1 if single else 0),
+                             _i32(_code(proj.dtype)), _stream()), "short_conv")
+    if not single and count > 1:
+        _check(lib.tb_short_conv_state(_ptr(proj), _i64(proj.stride(0)), _ptr(in_bias), _ptr(state), _ptr(row_start),
+                                       _ptr(seq_begin), _ptr(state_slots), _i32(num_seqs), _i32(channels), _i32(count),
+                                       _i32(_code(proj.dtype)), _stream()), "short_conv_state")
+    return out
+
+
+def _rglru_vectors(width: int, *vectors: torch.Tensor) -> None:
+    _cuda(*vectors)
+    for v in vectors:
+        _need(v.dtype == torch.float32 and v.numel() == width and v.is_contiguous(), "rglru vectors are float32 [width]")
+
+
+def rglru_step(u: torch.Tensor, weight: torch.Tensor, bias_r: torch.Tensor, bias_i: torch.Tensor, rate: torch.Tensor,
+               y: torch.Tensor, y_bias: torch.Tensor, state: torch.Tensor, state_slots: torch.Tensor,
+               out: torch.Tensor) -> torch.Tensor:
+    """One step of the recurrence for every row of ``u`` (row ``t`` belongs to the request in slot ``state_slots[t]``, no
+    slot twice): see :func:`rglru`."""
+    rows, width = u.shape
+    blocks, _, size = weight.shape
+    _cuda(u, weight, y, state, state_slots, out)
+    _rglru_vectors(width, bias_r, bias_i, rate, y_bias)
+    _need(u.stride(1) == 1 and weight.is_contiguous() and weight.dtype == u.dtype and tuple(weight.shape) == (blocks, 2 * size, size)
+          and blocks * size == width, "rglru u/weight")
+    _need(y.stride(1) == 1 and out.stride(1) == 1 and y.dtype == out.dtype == u.dtype and tuple(y.shape) == tuple(out.shape) == (rows, width),
+          "rglru y/out")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == width and state_slots.dtype == torch.int32
+          and state_slots.numel() >= rows, "rglru state")
+    lib = load_library("rglru")
+    _check(lib.tb_rglru_gates(_ptr(u), _i64(u.stride(0)), _ptr(weight), _ptr(bias_r), _ptr(bias_i), _ptr(rate), _ptr(None),
+                              _ptr(state), _ptr(state_slots), _ptr(y), _i64(y.stride(0)), _ptr(y_bias), _ptr(out),
+                              _i64(out.stride(0)), _i32(rows), _i32(blocks), _i32(size), _i32(_code(u.dtype)), _stream()),
+           "rglru_step")
+    return out
+
+
+def rglru_gates(u: torch.Tensor, weight: torch.Tensor, bias_r: torch.Tensor, bias_i: torch.Tensor, rate: torch.Tensor,
+                pairs: torch.Tensor) -> torch.Tensor:
+    """``pairs[t, c] = (a, sqrt(1 - a^2) i u)`` (float32 ``[T, width, 2]``), ``log a = rate * r``: see :func:`rglru`."""
+    rows, width = u.shape
+    blocks, _, size = weight.shape
+    _cuda(u, weight, pairs)
+    _rglru_vectors(width, bias_r, bias_i, rate)
+    _need(u.stride(1) == 1 and weight.is_contiguous() and weight.dtype == u.dtype and tuple(weight.shape) == (blocks, 2 * size, size)
+          and blocks * size == width, "rglru u/weight")
+    _f32_rows(pairs, (rows, width, 2), "rglru pairs are contiguous float32 [T, width, 2]")
+    lib = load_library("rglru")
+    none = _ptr(None)
+    _check(lib.tb_rglru_gates(_ptr(u), _i64(u.stride(0)), _ptr(weight), _ptr(bias_r), _ptr(bias_i), _ptr(rate), _ptr(pairs),
+                              none, none, none, _i64(0), none, none, _i64(0), _i32(rows), _i32(blocks), _i32(size),
+                              _i32(_code(u.dtype)), _stream()), "rglru_gates")
+    return pairs
+
+
+def rglru_scan(pairs: torch.Tensor, y: torch.Tensor, y_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+               row_start: torch.Tensor, state_slots: torch.Tensor, *, num_seqs: int, max_new: int) -> torch.Tensor:
+    """``S_t = a_t S_(t-1) + x_t`` over the pairs of every sequence, ``out = S * gelu_tanh(y + y_bias)``; ``state`` float32
+    ``[slots, width]`` is read and renewed: see :func:`rglru`."""
+    rows, width = out.shape
+    _cuda(pairs, y, state, out, row_start, state_slots)
+    _rglru_vectors(width, y_bias)
+    _f32_rows(pairs, (rows, width, 2), "rglru pairs are contiguous float32 [T, width, 2]")
+    _need(y.stride(1) == 1 and out.stride(1) == 1 and y.dtype == out.dtype and tuple(y.shape) == (rows, width), "rglru y/out")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == width, "rglru state")
+    _need(row_start.dtype == torch.int32 and state_slots.dtype == torch.int32, "rglru metadata must be int32")
+    lib = load_library("rglru")
+    _check(lib.tb_rglru_scan(_ptr(pairs), _ptr(y), _i64(y.stride(0)), _ptr(y_bias), _ptr(state), _ptr(out), _i64(out.stride(0)),
+                             _ptr(row_start), _ptr(state_slots), _i32(num_seqs), _i32(width), _i32(max_new),
+                             _i32(_code(out.dtype)), _stream()), "rglru_scan")
+    return out
+
+
+def rglru(u: torch.Tensor, weight: torch.Tensor, bias_r: torch.Tensor, bias_i: torch.Tensor, rate: torch.Tensor,
+          y: torch.Tensor, y_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor, row_start: torch.Tensor,
+          state_slots: torch.Tensor, *, num_seqs: int, max_new: int) -> torch.Tensor:
+    """The real-gated linear recurrent unit over ``u`` ``[T, width]``: with ``r, i`` the sigmoids of a square matrix per block
+    of channels (``weight`` ``[blocks, 2 S, S]``, rows alternating r, i) and a bias, ``log a = rate * r``, ``S_t = a S_(t-1) +
+    sqrt(1 - a^2) i u`` and ``out = S * gelu_tanh(y + y_bias)``.  One launch where every sequence brings one row, else the
+    gates and the scan."""
+    if max_new == 1 and num_seqs == u.shape[0]:
+        return rglru_step(u, weight, bias_r, bias_i, rate, y, y_bias, state, state_slots, out)
+    pairs = torch.empty((u.shape[0], u.shape[1], 2), dtype=torch.float32, device=u.device)
+    rglru_gates(u, weight, bias_r, bias_i, rate, pairs)
+    return rglru_scan(pairs, y, y_bias, state, out, row_start, state_slots, num_seqs=num_seqs, max_new=max_new)
 
 
 # ----------------------------------------------------------------------------- blocks whose two branches read one stream
@@ -989,12 +1113,14 @@ def sum_concat(residual: torch.Tensor, update_a: Optional[torch.Tensor], update_
     return out
 
 
-ACT_SILU, ACT_GELU_TANH = 0, 1
+ACT_SILU, ACT_GELU_TANH, ACT_CLAMPED = 0, 1, 2
 
 
-def gated_activation(gate_up: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, activation: int) -> torch.Tensor:
+def gated_activation(gate_up: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, activation: int,
+                     limit: float = 0.0, slope: float = 0.0) -> torch.Tensor:
     """``out = act(gate + bias[:I]) * (up + bias[I:])``; gate and up are the two halves of ``gate_up``'s rows, ``bias``
-    (float32 ``[2 I]``) may be None; ``activation``: ``ACT_SILU`` or ``ACT_GELU_TANH``."""
+    (float32 ``[2 I]``) may be None; ``activation``: ``ACT_SILU`` or ``ACT_GELU_TANH``, or ``ACT_CLAMPED``, which clamps
+    both halves: ``g * sigmoid(slope * g) * (u + 1)`` with ``g = min(gate, limit)``, ``u = min(max(up, -limit), limit)``."""
     _cuda(gate_up, bias, out)
     rows, inter = out.shape
     _need(gate_up.stride(1) == 1 and gate_up.shape == (rows, 2 * inter) and out.stride(1) == 1
@@ -1003,8 +1129,8 @@ def gated_activation(gate_up: torch.Tensor, bias: Optional[torch.Tensor], out: t
           "gated_activation bias")
     lib = load_library("pointwise")
     _check(lib.tb_gated_activation(_ptr(gate_up), _i64(gate_up.stride(0)), _ptr(bias), _ptr(out), _i64(out.stride(0)),
-                                   _i32(rows), _i32(inter), _i32(activation), _i32(_code(out.dtype)), _stream()),
-           "gated_activation")
+                                   _i32(rows), _i32(inter), _i32(activation), _f32(limit), _f32(slope),
+                                   _i32(_code(out.dtype)), _stream()), "gated_activation")
     return out
 
 
@@ -1107,13 +1233,27 @@ def rope_norm_cache(proj: torch.Tensor, q_out: torch.Tensor, cache: torch.Tensor
                     seq_of_row: torch.Tensor, block_table: torch.Tensor, inv_freq: Optional[torch.Tensor], *,
                     amplitude: float, heads: int, kv_heads: int, dim: int, vdim: int, rot_dims: int,
                     unit_norm: bool, eps: float, page_size: int, write_kv: bool = True,
-                    bias: Optional[torch.Tensor] = None) -> None:
+                    bias: Optional[torch.Tensor] = None, leave_values: Optional[torch.Tensor] = None,
+                    mix_values=None) -> None:
     """With ``bias`` (float32, as wide as the projected row) the projections' biases are added first.  Rotate-half rotation of the first ``rot_dims`` numbers of every query and key head of ``proj`` (cosine and sine
     times ``amplitude``), then, with ``unit_norm``, every head over ``sqrt(mean(head^2) + eps)``; queries into ``q_out``,
-    keys and values into the pages of ``cache`` (``[kv_heads, page, dim]`` keys then ``[kv_heads, page, vdim]`` values)."""
+    keys and values into the pages of ``cache`` (``[kv_heads, page, dim]`` keys then ``[kv_heads, page, vdim]`` values).
+    ``leave_values`` (float32 ``[T, kv_heads * vdim]``) receives the values as well; ``mix_values = (first, mix)``, such rows
+    of an earlier layer and one float32 number on the device: ``(1 - mix) * v + mix * first`` is stored instead of ``v``."""
     _cuda(proj, q_out, cache, positions, seq_of_row, block_table, inv_freq)
     rows = q_out.shape[0]
     channels = heads * dim + kv_heads * (dim + vdim)
+    _need(leave_values is None or mix_values is None, "rope_norm_cache: values are left or mixed, not both")
+    value_mode, first, mix = 0, None, None
+    if leave_values is not None:
+        value_mode, first = 1, leave_values
+    elif mix_values is not None:
+        value_mode, (first, mix) = 2, mix_values
+        _cuda(mix)
+        _need(mix.dtype == torch.float32 and mix.numel() == 1, "rope_norm_cache mix is one float32 number")
+    if first is not None:
+        _cuda(first)
+        _f32_rows(first, (rows, kv_heads * vdim), "rope_norm_cache values of the first layer")
     _need(proj.stride(1) == 1 and proj.shape[1] >= channels and proj.shape[0] == rows, "rope_norm_cache proj")
     _need(q_out.stride(1) == 1 and q_out.shape[1] == heads * dim and q_out.dtype == proj.dtype, "rope_norm_cache q_out")
     _need(cache.dtype == proj.dtype and cache.is_contiguous(), "rope_norm_cache cache dtype")
@@ -1130,7 +1270,8 @@ def rope_norm_cache(proj: torch.Tensor, q_out: torch.Tensor, cache: torch.Tensor
                                   _ptr(positions), _ptr(seq_of_row), _ptr(block_table), _i32(block_table.stride(0)),
                                   _ptr(inv_freq), _ptr(bias), _f32(amplitude), _i32(rows), _i32(heads), _i32(kv_heads), _i32(dim),
                                   _i32(vdim), _i32(rot_dims), _i32(1 if unit_norm else 0), _f32(eps), _i32(page_size),
-                                  _i32(1 if write_kv else 0), _i32(_code(proj.dtype)), _stream()), "rope_norm_cache")
+                                  _i32(1 if write_kv else 0), _i32(value_mode), _ptr(first), _ptr(mix),
+                                  _i32(_code(proj.dtype)), _stream()), "rope_norm_cache")
 
 
 def pool_blocks(cache: torch.Tensor, pool_cache: torch.Tensor, positions: torch.Tensor, seq_of_row: torch.Tensor,
@@ -1153,7 +1294,7 @@ def pool_blocks(cache: torch.Tensor, pool_cache: torch.Tensor, positions: torch.
 
 # ----------------------------------------------------------------------------- routed experts
 
-EXPERT_PLAIN, EXPERT_SQUARED_RELU = 0, 1
+EXPERT_PLAIN, EXPERT_SQUARED_RELU, EXPERT_GATED_CLAMPED = 0, 1, 2
 
 
 def choose_topk(logits: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor) -> None:
@@ -1187,6 +1328,20 @@ def choose_grouped(logits: torch.Tensor, ids: torch.Tensor, weights: torch.Tenso
                                  _i32(keep), _f32(weight_scale), _stream()), "choose_grouped")
 
 
+def choose_sigmoid(logits: torch.Tensor, experts: int, ids: torch.Tensor, weights: torch.Tensor) -> None:
+    """The ``top`` largest of the first ``experts`` numbers of every row of ``logits`` (float32; largest first, the lowest
+    index among equals) into ``ids`` and their sigmoids, each on its own, into ``weights``."""
+    _cuda(logits, ids, weights)
+    rows, top = ids.shape
+    _need(logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[0] == rows and logits.shape[1] >= experts,
+          "choose_sigmoid logits")
+    _need(ids.dtype == torch.int32 and ids.is_contiguous() and weights.dtype == torch.float32 and weights.is_contiguous()
+          and tuple(weights.shape) == (rows, top), "choose_sigmoid ids/weights")
+    lib = load_library("experts")
+    _check(lib.tb_choose_sigmoid(_ptr(logits), _i64(logits.stride(0)), _ptr(ids), _ptr(weights), _i32(rows), _i32(experts),
+                                 _i32(top), _stream()), "choose_sigmoid")
+
+
 def expert_plan(ids: torch.Tensor, experts: int, offsets: torch.Tensor, order: torch.Tensor) -> None:
     """Group the assignments ``ids.flatten()`` by expert: ``order[offsets[e] : offsets[e + 1]]`` are expert ``e``'s."""
     _cuda(ids, offsets, order)
@@ -1204,14 +1359,26 @@ def expert_linear_tensor_cores(dtype: torch.dtype, in_features: int) -> bool:
 
 
 def expert_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, order: torch.Tensor,
-                  *, source_div: int, epilogue: int = EXPERT_PLAIN) -> torch.Tensor:
+                  *, source_div: int, epilogue: int = EXPERT_PLAIN, row_weights: Optional[torch.Tensor] = None,
+                  limit: float = 0.0, slope: float = 0.0) -> torch.Tensor:
     """``out[a] = act(weight[expert(a)] @ x[a // source_div])`` for every assignment ``a`` (``weight`` ``[E, N, K]``,
-    ``out`` ``[assignments, N]`` in ``x``'s dtype or float32), grouped as ``expert_plan`` left them."""
+    ``out`` ``[assignments, N]`` in ``x``'s dtype or float32), grouped as ``expert_plan`` left them.
+    ``EXPERT_GATED_CLAMPED``: the weight's rows alternate (gate, up) and ``out`` is ``[assignments, N / 2]``: with ``G`` and
+    ``U`` the two sums times the assignment's number in ``row_weights`` (float32, or None), ``g = min(G, limit)``, ``u =
+    min(max(U, -limit), limit)``: ``g * sigmoid(slope * g) * (u + 1)``."""
     _cuda(x, weight, out, offsets, order)
     experts, n, k = weight.shape
     count = out.shape[0]
     _need(x.stride(1) == 1 and x.shape[1] == k and weight.is_contiguous() and weight.dtype == x.dtype, "expert_linear x/weight")
-    _need(out.stride(1) == 1 and out.shape[1] == n and out.dtype in (x.dtype, torch.float32), "expert_linear out")
+    gated = epilogue == EXPERT_GATED_CLAMPED
+    _need(out.stride(1) == 1 and out.shape[1] == (n // 2 if gated else n) and out.dtype in (x.dtype, torch.float32),
+          "expert_linear out")
+    _need(not gated or n % 2 == 0, "expert_linear: a gated weight has an even number of rows")
+    _need(row_weights is None or gated, "expert_linear: only the gated form weighs its input")
+    if row_weights is not None:
+        _cuda(row_weights)
+        _need(row_weights.dtype == torch.float32 and row_weights.is_contiguous() and row_weights.numel() == count,
+              "expert_linear row weights")
     _need(order.numel() == count and offsets.numel() == experts + 1, "expert_linear plan")
     _need(x.shape[0] * source_div >= count, "expert_linear: sources do not cover the assignments")
     tensor_cores = (expert_linear_tensor_cores(x.dtype, k) and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
@@ -1219,23 +1386,31 @@ def expert_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, offs
     lib = load_library("experts")
     _check(lib.tb_expert_linear(_ptr(x), _i64(x.stride(0)), _ptr(weight), _ptr(out), _i64(out.stride(0)), _ptr(offsets),
                                 _ptr(order), _i32(count), _i32(experts), _i32(source_div), _i32(n), _i32(k),
-                                _i32(epilogue), _i32(_code(x.dtype)), _i32(_code(out.dtype)),
+                                _i32(epilogue), _ptr(row_weights), _f32(limit), _f32(slope), _i32(_code(x.dtype)),
+                                _i32(_code(out.dtype)),
                                 _i32(1 if tensor_cores else 0), _stream()), "expert_linear")
     return out
 
 
-def expert_combine(y: torch.Tensor, weights: torch.Tensor, base: Optional[torch.Tensor], out: torch.Tensor) -> torch.Tensor:
-    """``out[t] = (base[t] if base is given else 0) + sum_s weights[t, s] * y[t * top + s]``, all float32."""
-    _cuda(y, weights, base, out)
+def expert_combine(y: torch.Tensor, weights: Optional[torch.Tensor], base: Optional[torch.Tensor], out: torch.Tensor,
+                   base_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[t] = (base[t] if base is given else 0) + sum_s weights[t, s] * y[t * top + s]``, all float32; without ``weights``
+    the slots are added as they are.  ``base_gate`` (float32, a number per row at any stride): the base is multiplied by
+    its sigmoid."""
+    _cuda(y, weights, base, out, base_gate)
     rows, width = out.shape
-    top = weights.shape[1]
+    top = weights.shape[1] if weights is not None else (y.shape[0] // rows if rows else 1)
     _f32_rows(y, (rows * top, width), "expert_combine y")
     _f32_rows(weights, (rows, top), "expert_combine weights")
     _f32_rows(base, (rows, width), "expert_combine base")
     _f32_rows(out, (rows, width), "expert_combine out")
+    if base_gate is not None:
+        _need(base is not None and base_gate.dtype == torch.float32 and base_gate.dim() == 1 and base_gate.numel() == rows,
+              "expert_combine base gate")
     lib = load_library("experts")
-    _check(lib.tb_expert_combine(_ptr(y), _ptr(weights), _ptr(base), _ptr(out), _i32(rows), _i32(width), _i32(top),
-                                 _stream()), "expert_combine")
+    _check(lib.tb_expert_combine(_ptr(y), _ptr(weights), _ptr(base), _ptr(base_gate),
+                                 _i64(base_gate.stride(0) if base_gate is not None else 0), _ptr(out), _i32(rows), _i32(width),
+                                 _i32(top), _stream()), "expert_combine")
     return out
 
 
@@ -1248,8 +1423,9 @@ def norm_add_norm(residual: torch.Tensor, update: Optional[torch.Tensor], post, 
                   out: Optional[torch.Tensor], copy: Optional[torch.Tensor], eps: float) -> None:
     """``residual += post(update)`` (32-bit, in place; without ``update`` the stream stays), then ``out =
     following(residual)`` and ``copy = residual``, both rounded once to their dtype.  ``post`` and ``following`` are
-    ``None`` or ``(kind, weight, bias)`` with kind ``NORM_LAYER`` (``(v - mean) / sqrt(var + eps) * weight + bias``) or
-    ``NORM_RMS`` (``v / sqrt(mean(v^2) + eps) * weight``, bias None); both use ``eps``."""
+    ``None`` or ``(kind, weight, bias[, groups])`` with kind ``NORM_LAYER`` (``(v - mean) / sqrt(var + eps) * weight + bias``)
+    or ``NORM_RMS`` (``v / sqrt(mean(v^2) + eps) * weight`` over each of ``groups`` equal consecutive parts of the
+    row, bias None); both use ``eps``."""
     _cuda(residual, update, out, copy)
     rows, width = residual.shape
     _f32_rows(residual, (rows, width), "norm_add_norm: the stream is contiguous float32")
@@ -1264,21 +1440,42 @@ def norm_add_norm(residual: torch.Tensor, update: Optional[torch.Tensor], post, 
 
     def parts(norm):
         if norm is None:
-            return NORM_NONE, None, None
-        kind, weight, bias = norm
+            return NORM_NONE, None, None, 1
+        kind, weight, bias, *rest = norm
+        groups = rest[0] if rest else 1
         _need(kind in (NORM_LAYER, NORM_RMS), "norm_add_norm: unknown norm kind")
         for v in (weight, bias):
             _need(v is None or (v.is_cuda and v.dtype == torch.float32 and v.numel() == width and v.is_contiguous()),
                   "norm_add_norm weight/bias")
         _need(weight is not None and (kind != NORM_LAYER or bias is not None), "norm_add_norm: a norm needs its vectors")
-        return kind, weight, bias
+        _need(groups >= 1 and width % groups == 0 and (groups == 1 or kind == NORM_RMS), "norm_add_norm groups")
+        return kind, weight, bias, groups
 
-    post_kind, post_w, post_b = parts(post)
-    next_kind, next_w, next_b = parts(following)
+    post_kind, post_w, post_b, post_groups = parts(post)
+    next_kind, next_w, next_b, next_groups = parts(following)
     lib = load_library("sandwich_norm")
     _check(lib.tb_norm_add_norm(_ptr(residual), _ptr(update), _i32(post_kind), _ptr(post_w), _ptr(post_b), _i32(next_kind),
                                 _ptr(next_w), _ptr(next_b), _ptr(out), _ptr(copy), _i32(rows), _i32(width), _f32(eps),
-                                _i32(_code(dtype) if dtype is not None else 0), _stream()), "norm_add_norm")
+                                _i32(post_groups), _i32(next_groups), _i32(_code(dtype) if dtype is not None else 0), _stream()), "norm_add_norm")
+
+
+def embedding_norm(tokens: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, position_table: torch.Tensor,
+                   weight: torch.Tensor, groups: int, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """``out[t] = rms(float32(table[tokens[t]]) + float32(position_table[positions[t]])) * weight`` over ``groups`` equal
+    consecutive parts of the row; ``out`` and ``weight`` float32, the tables in the run dtype."""
+    _cuda(tokens, positions, table, position_table, weight, out)
+    rows, width = out.shape
+    _f32_rows(out, (rows, width), "embedding_norm out is contiguous float32")
+    for t in (tokens, positions):
+        _need(t.dtype == torch.int32 and t.is_contiguous() and t.numel() >= rows, "embedding_norm tokens and positions are int32")
+    _need(table.is_contiguous() and position_table.is_contiguous() and table.dtype == position_table.dtype
+          and table.shape[1] == width == position_table.shape[1], "embedding_norm tables")
+    _need(weight.dtype == torch.float32 and weight.numel() == width and weight.is_contiguous(), "embedding_norm weight")
+    lib = load_library("sandwich_norm")
+    _check(lib.tb_embedding_norm(_ptr(tokens), _ptr(positions), _ptr(table), _ptr(position_table), _ptr(weight), _ptr(out),
+                                 _i32(rows), _i32(width), _i32(table.shape[0]), _i32(position_table.shape[0]), _i32(groups),
+                                 _f32(eps), _i32(_code(table.dtype)), _stream()), "embedding_norm")
+    return out
 
 
 def gated_rms_norm(v: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, eps: float) -> torch.Tensor:

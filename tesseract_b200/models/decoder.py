@@ -121,18 +121,25 @@ class DecoderModel:
         return needs
 
     # ------------------------------------------------------------------ forward
+    def _embed(self, ctx: StepContext) -> torch.Tensor:
+        token_ids = ctx.token_ids[:ctx.num_rows]
+        if self.embedding.takes_positions:
+            return self.embedding.forward(token_ids, positions=ctx.positions[:ctx.num_rows])
+        return self.embedding.forward(token_ids)
+
     def forward(self, ctx: StepContext, bindings: Sequence[Optional[CacheBinding]],
                 want_rows: Optional[torch.Tensor], want_every_row: bool = False) -> Optional[torch.Tensor]:
         """Run the step's rows; return float32 logits ``[len(want_rows), vocab]`` or ``None``.
         ``want_every_row``: the caller knows that ``want_rows`` is ``0 .. num_rows - 1`` (a decode step), so the
         rows need not be gathered before the head."""
-        hidden = self.embedding.forward(ctx.token_ids[:ctx.num_rows])
+        ctx.carried.clear()
+        hidden = self._embed(ctx)
         stream = ResidualStream(hidden, None)
         order = self.spec.run_order
         # the embedding output that injections read: rows of their own, since blocks add into the stream in place
         origin = None
         if any(injection.reads_origin for injection in self.injections):
-            origin = self.embedding.forward(ctx.token_ids[:ctx.num_rows])
+            origin = self._embed(ctx)
         wants_logits = want_rows is not None and want_rows.numel() > 0
         every_row = wants_logits and want_every_row and want_rows.numel() == ctx.num_rows
         for index, entry in enumerate(order):
@@ -143,9 +150,10 @@ class DecoderModel:
                 stream = block.forward(stream, ctx, bindings[index])
                 continue
             # the norm that will consume what this block returns: the next block's first one, or the final norm if
-            # it runs on every row (on a few wanted rows it runs after they have been picked out)
+            # it runs on every row (on a few wanted rows it runs after they have been picked out); None where an
+            # injection changes the stream in between
             if index + 1 < len(order):
-                next_norm = self.layers[order[index + 1].layer].entry_norm()
+                next_norm = self.layers[order[index + 1].layer].entry_norm() if order[index + 1].inject is None else None
             else:
                 next_norm = self.final_norm if every_row else None
             stream = block.forward(stream, ctx, bindings[index], next_norm=next_norm)

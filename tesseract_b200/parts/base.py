@@ -24,7 +24,8 @@ Kinds and what each must provide:
     arranges norms, mixer and feed-forward: ``forward(stream, ctx, cache)`` on a
     :class:`ResidualStream`.
 ``Embedding`` / ``Head``
-    ``forward(token_ids)`` -> ``[T, hidden]`` / ``forward(x)`` -> float32 ``[S, vocab]``.
+    ``forward(token_ids)`` (``forward(token_ids, positions=...)`` if it says ``takes_positions``) -> ``[T, hidden]`` /
+    ``forward(x)`` -> float32 ``[S, vocab]``.
 ``Injection``
     ``forward(stream, origin, ctx)`` -> the new :class:`ResidualStream`: a step between two blocks that mixes the
     stream with the embedding output.
@@ -133,6 +134,9 @@ class PagedNeed:
     # positions says P: its pages fill P times as slowly and its pool is that much smaller)
     positions_per_entry: int = 1
 
+    # the first positions of a request that every later query still reads, whatever the window: their pages stay
+    keep_first: int = 0
+
     def page_shape(self, page_size: int) -> Tuple[int, ...]:
         raise NotImplementedError
 
@@ -193,6 +197,8 @@ class PagedKeyValueNeed(PagedNeed):
     # is still being filled stay although the window has passed them (a later step reads them once more, to average
     # the finished run, say)
     hold: Optional[int] = None
+    # with a window: the first positions of the sequence that every later token still sees
+    keep_first: int = 0
 
     def page_shape(self, page_size: int) -> Tuple[int, ...]:
         value_heads = self.num_kv_heads if self.num_value_heads is None else self.num_value_heads
@@ -305,6 +311,8 @@ class StepContext:
     host_slots: Sequence[int] = ()
     max_new: int = 1
     max_context: int = 1
+    # what a part leaves for parts of later layers of the same step (rows of the step, by name)
+    carried: Dict[str, torch.Tensor] = field(default_factory=dict)
 
     @property
     def decode_only(self) -> bool:
@@ -471,6 +479,8 @@ class FeedForward(Part):
 
 
 class Embedding(Part):
+    takes_positions = False      # True if ``forward`` also takes ``positions`` (int32, one per token)
+
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
 

@@ -30,7 +30,9 @@ sum and both norms are one kernel.  A layer without a feed-forward leaves (x, a)
     x <- x + token_input(x, tokens)                                     (absent without a token input)
 
 The norm of a sublayer's result, the addition and the norm in front of the next sublayer are one kernel
-(``norm_add_norm``); it also leaves the rounded stream that the token input's first product reads.
+(``norm_add_norm``); it also leaves the rounded stream that the token input's first product reads.  Where a layer has no
+token input, the kernel behind its last sublayer also takes the norm that consumes the stream next (the next block's
+first norm, or the final norm).
 
 ``gated_pre_norm`` is the pre-norm arrangement over a 32-bit stream in which every sublayer's result is weighted, feature
 by feature, by a learned scale and by a gate that reads the sublayer's own input:
@@ -119,9 +121,13 @@ class ParallelBlock(Block):
         return x_mixer, (second.forward(residual) if second is not None else None)
 
     def forward(self, stream: ResidualStream, ctx: StepContext, cache: Optional[CacheBinding]) -> ResidualStream:
-        if stream.prepared is not None:
+        if stream.prepared is not None and stream.prepared.norm is not self.norms["mixer"]:
             raise NotImplementedError("a parallel block takes the stream as a residual and its pending updates")
-        x_mixer, x_feed = self._norms_of_sum(stream)
+        if stream.prepared is not None:               # the block in front took the mixer's norm with its last addition
+            x_mixer = stream.prepared.materialize()
+            x_feed = self.norms["feed_forward"].forward(stream.residual) if self.feed_forward is not None else None
+        else:
+            x_mixer, x_feed = self._norms_of_sum(stream)
         mixed = self.mixer.forward(x_mixer, ctx, cache)
         if self.feed_forward is None:
             return ResidualStream(stream.residual, mixed)
@@ -134,6 +140,7 @@ class SandwichBlock(Block):
     Every norm offers ``norm_parameters()`` (what ``kernels.norm_add_norm`` takes) and ``eps``; all share one ``eps``."""
 
     accepts_token_input = True
+    accepts_next_norm = True
 
     def __init__(self, norms, mixer, feed_forward, token_input=None):
         super().__init__(norms, mixer, feed_forward)
@@ -153,12 +160,13 @@ class SandwichBlock(Block):
     def entry_norm(self) -> Optional[Norm]:
         return self.norms["pre_mixer"]
 
-    def forward(self, stream: ResidualStream, ctx: StepContext, cache) -> ResidualStream:
+    def forward(self, stream: ResidualStream, ctx: StepContext, cache, next_norm: Optional[Norm] = None) -> ResidualStream:
         import torch
 
         from .. import kernels
 
-        if stream.prepared is not None or stream.update_b is not None:
+        prepared = stream.prepared
+        if (prepared is not None and prepared.norm is not self.norms["pre_mixer"]) or stream.update_b is not None:
             raise NotImplementedError("a sandwich block takes the stream as a residual and at most one pending update")
         residual = stream.residual
         if residual.dtype != torch.float32:
@@ -168,8 +176,11 @@ class SandwichBlock(Block):
         def rows_like():
             return torch.empty(residual.shape, dtype=dtype, device=residual.device)
 
-        x = rows_like()
-        kernels.norm_add_norm(residual, stream.update, None, self.norms["pre_mixer"].norm_parameters(), x, None, self.eps)
+        if prepared is not None:
+            x = prepared.materialize()                    # the block in front took this norm with its last addition
+        else:
+            x = rows_like()
+            kernels.norm_add_norm(residual, stream.update, None, self.norms["pre_mixer"].norm_parameters(), x, None, self.eps)
         mixed = self.mixer.forward(x, ctx, cache)
         wants_copy = self.token_input is not None and dtype != torch.float32
         if self.feed_forward is not None:
@@ -179,6 +190,13 @@ class SandwichBlock(Block):
             update, post = self.feed_forward.forward(x, ctx), self.norms["post_feed_forward"]
         else:
             update, post = mixed, self.norms["post_mixer"]
+        following = None
+        if self.token_input is None and hasattr(next_norm, "norm_parameters") and next_norm.eps == self.eps:
+            following = next_norm
+        if following is not None:
+            rows = rows_like()
+            kernels.norm_add_norm(residual, update, post.norm_parameters(), following.norm_parameters(), rows, None, self.eps)
+            return ResidualStream(residual, None, prepared=FinishedNorm(following, residual, rows))
         copy = rows_like() if wants_copy else None
         kernels.norm_add_norm(residual, update, post.norm_parameters(), None, None, copy, self.eps)
         if self.token_input is not None:

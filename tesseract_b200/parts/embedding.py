@@ -58,6 +58,46 @@ class TokenEmbedding(Embedding):
         return kernels.embedding(token_ids, self.table, out)
 
 
+@EMBEDDINGS.register("positioned_embedding")
+class PositionedEmbedding(Embedding):
+    """A token's row plus a learned row for its position, normed: ``rms(table[token] + positions[p]) * weight`` over
+    ``groups`` equal consecutive parts of the row, as the 32-bit start of a residual stream kept in 32-bit.
+
+    params: ``vocab_size, hidden_size, max_positions, groups, eps``; weights: ``table``, ``positions``, ``weight``."""
+
+    graph_safe = True
+    takes_positions = True
+
+    def __init__(self, spec: PartSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
+        super().__init__(spec, tensors, runtime)
+        p = spec.params
+        self.hidden_size = int(p["hidden_size"])
+        self.groups = int(p.get("groups") or 1)
+        self.eps = float(p["eps"])
+        if self.groups < 1 or self.hidden_size % self.groups:
+            raise ValueError(f"a norm over {self.groups} groups needs a size that they divide, got {self.hidden_size}")
+        self.table = runtime.matrix(tensors["table"])
+        self.positions = runtime.matrix(tensors["positions"])
+        self.weight = runtime.vector_f32(tensors["weight"])
+
+    @classmethod
+    def expected_tensors(cls, spec: PartSpec) -> Dict[str, ExpectedTensor]:
+        p, w = spec.params, spec.weights
+        hidden = int(p["hidden_size"])
+        return {w["table"]: ExpectedTensor((int(p["vocab_size"]), hidden)),
+                w["positions"]: ExpectedTensor((int(p["max_positions"]), hidden)), w["weight"]: ExpectedTensor((hidden,))}
+
+    @classmethod
+    def random_tensor(cls, spec, role, shape, generator) -> torch.Tensor:
+        noise = torch.randn(shape, generator=generator, dtype=torch.float32)
+        return 1.0 + noise * 0.1 if role == "weight" else noise * (0.3 if role == "positions" else 1.0)
+
+    def forward(self, token_ids: torch.Tensor, positions: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if out is None:
+            out = torch.empty((token_ids.numel(), self.hidden_size), dtype=torch.float32, device=self.table.device)
+        return kernels.embedding_norm(token_ids, positions, self.table, self.positions, self.weight, self.groups, self.eps, out)
+
+
 @HEADS.register("lm_head")
 class LMHead(Head):
     """params: ``vocab_size, hidden_size``, optional ``scale`` (the logits are multiplied by it); weights: ``weight``.

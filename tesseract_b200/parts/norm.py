@@ -96,6 +96,10 @@ class GroupedRMSNorm(Norm):
         norms of the same row with the same ``eps`` differ in their weights only and may leave one kernel together."""
         return (self.weight, self.eps) if self.groups == 1 else None
 
+    def norm_parameters(self):
+        """``(kind, weight, bias, groups)`` as ``kernels.norm_add_norm`` takes a norm."""
+        return (kernels.NORM_RMS, self.weight, None, self.groups)
+
     def forward_sum(self, residual: torch.Tensor, update_a: Optional[torch.Tensor], update_b: Optional[torch.Tensor],
                     out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``residual += update_a + update_b`` (either may be None; 32-bit, in place), then the norm of the sum."""

@@ -13,9 +13,14 @@ Per row ``h`` (the mixer's input):
   from position ``p`` if ``(b + 1) * pool <= p - size + 1``), one key and one value that are the averages of the block's
   keys and values as the pages hold them; so for up to ``pool - 1`` steps a token is visible neither by itself nor through
   its block.  The averages live in pages of their own (an entry a block) and are written by the step that brings a
-  block's last token.  Scores ``(q . k) * scale``, with ``softcap`` then ``softcap * tanh(score / softcap)``, the softmax
-  and the weights are 32-bit; with ``sink`` the denominator also holds ``exp`` of a learned number per query head;
-* with ``bias`` the three projections add a bias each;
+  block's last token.  A ``window`` may also keep the first ``keep_first`` positions of the sequence, which every row goes
+  on seeing (their pages stay; older pages behind the window go back to the pool).  Scores ``(q . k) * scale``, with ``softcap`` then ``softcap * tanh(score / softcap)``, the softmax
+  and the weights are 32-bit; with ``sink`` the denominator also holds ``exp`` of a learned number per query head; with
+  ``distance_bias`` the score of the key ``n`` positions back loses ``w * ln(1 + r * n)``, two numbers per query head;
+* with ``bias`` the three projections add a bias each, with ``output_bias`` the output projection does;
+* values may be mixed across layers: a part with ``value_mix`` ``"first"`` leaves its values in the step
+  (``StepContext.carried``), a later one with ``"mix"`` stores ``(1 - x) v + x v_first`` instead of its own values ``v``, ``x``
+  one learned number (the first part's values of the same token are rows of the same step, so nothing is cached for it);
 * the output projection's result comes out in 32-bit for a residual stream kept in 32-bit (``stream`` = ``"float32"``).
 
 Rotation, normalisation and the cache write are one kernel; the attention kernel is the one the other mixers with
@@ -42,9 +47,11 @@ _MASKS = {"causal": kernels.MASK_CAUSAL, "window": kernels.MASK_WINDOW, "window_
 @MIXERS.register("normed_attention")
 class NormedAttention(Mixer):
     """params: ``hidden_size, num_heads, num_kv_heads, key_dim, value_dim, scale``, ``mask`` (``{"kind": "causal" |
-    "window" | "window_pooled", "size": n, "pool": P}``), ``qk_norm_eps`` (None: queries and keys stay as rotated),
-    optional ``softcap``, ``sink`` (bool), ``bias`` (bool), ``stream``.  weights: ``q, k, v, o``, with ``bias`` also
-    ``q_bias, k_bias, v_bias``, with ``sink`` also ``sink`` ``[num_heads]``.  children: ``position``."""
+    "window" | "window_pooled", "size": n, "pool": P, "keep_first": k}``), ``qk_norm_eps`` (None: queries and keys stay as
+    rotated), optional ``softcap``, ``sink`` (bool), ``bias`` (bool), ``output_bias`` (bool), ``distance_bias`` (bool),
+    ``value_mix`` (``"first"`` | ``"mix"``), ``stream``.  weights: ``q, k, v, o``, with ``bias`` also ``q_bias, k_bias,
+    v_bias``, with ``output_bias`` ``o_bias``, with ``sink`` ``sink`` ``[num_heads]``, with ``distance_bias`` ``distance_weight``
+    and ``distance_rate`` (``[num_heads]`` each), to mix ``value_mix`` (one number).  children: ``position``."""
 
     graph_safe = True      # reads only device-side metadata of the step (and its shape)
 
@@ -67,10 +74,22 @@ class NormedAttention(Mixer):
         self.pool = int(mask.get("pool") or 0)
         if self.mask_kind == "window_pooled" and self.pool < 1:
             raise ValueError("a 'window_pooled' mask needs a positive pool")
+        self.keep_first = int(mask.get("keep_first") or 0)
+        if self.keep_first < 0 or (self.keep_first and self.mask_kind != "window"):
+            raise ValueError("keep_first is a number of positions that a 'window' mask keeps")
         self.softcap = float(p.get("softcap") or 0.0)
         if self.softcap < 0.0:
             raise ValueError("softcap must not be negative")
         self.sinks = runtime.vector_f32(tensors["sink"]) if p.get("sink") else None
+        self.distance_bias = None
+        if p.get("distance_bias"):
+            if self.mask_kind == "window_pooled":
+                raise ValueError("averaged blocks have no distance: a distance bias goes with the other masks")
+            self.distance_bias = (runtime.vector_f32(tensors["distance_weight"]), runtime.vector_f32(tensors["distance_rate"]))
+        self.value_mix = p.get("value_mix")
+        if self.value_mix not in (None, "first", "mix"):
+            raise ValueError(f"value_mix is 'first', 'mix' or absent, got {self.value_mix!r}")
+        self.mix = runtime.vector_f32(tensors["value_mix"]).reshape(1) if self.value_mix == "mix" else None
         self.biased = bool(p.get("bias"))
         eps = p.get("qk_norm_eps")
         self.unit_norm = eps is not None
@@ -88,7 +107,7 @@ class NormedAttention(Mixer):
             self.in_bias = torch.cat([tensors["q_bias"], tensors["k_bias"], tensors["v_bias"]]).to(
                 device=runtime.device, dtype=torch.float32).contiguous()
         self.in_proj = Linear(torch.cat([tensors["q"], tensors["k"], tensors["v"]], dim=0), runtime)
-        self.o_proj = Linear(tensors["o"], runtime)
+        self.o_proj = Linear(tensors["o"], runtime, bias=tensors["o_bias"] if p.get("output_bias") else None)
         position_spec = spec.children.get("position") or PartSpec.make("none")
         self.position = POSITION_ENCODINGS.get(position_spec.kind)(position_spec, {}, runtime)
         if self.position.kind not in ("rotary_blend", "none"):
@@ -113,14 +132,22 @@ class NormedAttention(Mixer):
         if p.get("bias"):
             out.update({w["q_bias"]: ExpectedTensor((heads * d,)), w["k_bias"]: ExpectedTensor((kv * d,)),
                         w["v_bias"]: ExpectedTensor((kv * dv,))})
+        if p.get("output_bias"):
+            out[w["o_bias"]] = ExpectedTensor((hidden,))
         if p.get("sink"):
             out[w["sink"]] = ExpectedTensor((heads,))
+        if p.get("distance_bias"):
+            out.update({w["distance_weight"]: ExpectedTensor((heads,)), w["distance_rate"]: ExpectedTensor((heads,))})
+        if p.get("value_mix") == "mix":
+            out[w["value_mix"]] = ExpectedTensor(())
         return out
 
     @classmethod
     def random_tensor(cls, spec, role, shape, generator) -> torch.Tensor:
         if role.endswith("_bias"):
             return torch.randn(shape, generator=generator, dtype=torch.float32) * 0.3
+        if role in ("distance_weight", "distance_rate", "value_mix"):
+            return torch.rand(shape, generator=generator, dtype=torch.float32) * 0.5 + 0.1
         if role == "sink":
             return torch.randn(shape, generator=generator, dtype=torch.float32)
         return torch.randn(shape, generator=generator, dtype=torch.float32) * (shape[-1] ** -0.5)
@@ -139,7 +166,7 @@ class NormedAttention(Mixer):
                     PooledBlocksNeed(num_kv_heads=self.num_kv_heads, key_dim=self.key_dim, value_dim=self.value_dim,
                                      pool=self.pool))
         return PagedKeyValueNeed(num_kv_heads=self.num_kv_heads, key_dim=self.key_dim, value_dim=self.value_dim,
-                                 window=self.mask_size if self.mask_kind == "window" else None)
+                                 window=self.mask_size if self.mask_kind == "window" else None, keep_first=self.keep_first)
 
     def attention_choice(self, rows: int) -> str:
         """The attention kernel of a step of ``rows`` rows (all three know the cap, the learned sink and pooled blocks)."""
@@ -162,12 +189,23 @@ class NormedAttention(Mixer):
         proj = self.in_proj.forward(x)
         rows = proj.shape[0]
         q = torch.empty((rows, self.q_width), dtype=proj.dtype, device=proj.device)
+        across = {}
+        if self.value_mix == "first":
+            across["leave_values"] = torch.empty((rows, self.num_kv_heads * self.value_dim), dtype=torch.float32,
+                                                 device=proj.device)
+            ctx.carried["first_values"] = across["leave_values"]
+        elif self.value_mix == "mix":
+            first = ctx.carried.get("first_values")
+            if first is None or first.shape != (rows, self.num_kv_heads * self.value_dim):
+                raise RuntimeError("a mixer that mixes values needs an earlier layer's values of the same width in the step")
+            across["mix_values"] = (first, self.mix)
         kernels.rope_norm_cache(proj, q, cache.storage, ctx.positions, ctx.seq_of_row, group.block_table, self.inv_freq,
                                 amplitude=self.amplitude, heads=self.num_heads, kv_heads=self.num_kv_heads,
                                 dim=self.key_dim, vdim=self.value_dim, rot_dims=self.rot_dims,
                                 unit_norm=self.unit_norm, eps=self.qk_norm_eps, page_size=cache.page_size,
-                                bias=self.in_bias)
-        extras = {"sinks": self.sinks, "softcap": self.softcap}
+                                bias=self.in_bias, **across)
+        extras = {"sinks": self.sinks, "softcap": self.softcap, "keep_first": self.keep_first,
+                  "distance_bias": self.distance_bias}
         if pooled is not None:
             pool_table = ctx.groups[pooled.group].block_table
             kernels.pool_blocks(cache.storage, pooled.storage, ctx.positions, ctx.seq_of_row, group.block_table, pool_table,

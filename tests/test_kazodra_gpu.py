@@ -562,8 +562,8 @@ def test_every_layer_run_matches_plain(engines, folders, name, dtype):
     seen = []
     original = SandwichBlock.forward
 
-    def recording(self, stream, ctx, cache):
-        out = original(self, stream, ctx, cache)
+    def recording(self, stream, ctx, cache, next_norm=None):
+        out = original(self, stream, ctx, cache, next_norm=next_norm)
         assert out.update is None and out.residual.dtype == torch.float32
         seen.append(out.residual.double().cpu())
         return out
