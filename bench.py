@@ -664,7 +664,7 @@ def run_kernels(args):
 
 
 # ----------------------------------------------------------------------------- another design beside Llama
-# `--design revesun|pekodra|kazodra|ladedra`: prefill and decode of a model of that design at layer sizes like a real model's (random
+# `--design revesun|pekodra|kazodra|ladedra|rirulix`: prefill and decode of a model of that design at layer sizes like a real model's (random
 # weights), beside a Llama (and, for Pekodra, a Revesun: the other design with a 32-bit stream) of the same width, heads, head sizes, layer count and about as many weights a layer, measured the
 # same way; then the design's own kernels alone, against the bytes they must move.  The default workload is untouched.
 DESIGN_SIZES = {
@@ -802,6 +802,31 @@ def ladedra_config(size, layers):
             "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "layers": [parallel if i % 2 else latent for i in range(layers)]}
 
 
+RIRULIX_SIZES = {
+    # (attention layers have the heads of the models beside it; recurrent layers are as wide as the stream, in blocks of 256
+    # channels; every layer routes: a gated expert has three matrices where Pekodra's has two, as Ladedra's)
+    "1b": dict(window=512, keep=4, blocks=8, taps=4, experts=32, top=4, expert_ff=640, shared_ff=1408),
+    "3b": dict(window=512, keep=4, blocks=12, taps=4, experts=32, top=4, expert_ff=640, shared_ff=1408),
+    "8b": dict(window=512, keep=4, blocks=16, taps=4, experts=32, top=4, expert_ff=1408, shared_ff=2752),
+}
+
+
+def rirulix_config(size, layers):
+    """Even layers: window attention that keeps the first tokens, with a distance bias and values mixed with the first
+    layer's; odd layers: a real-gated linear recurrent unit.  Every layer routes to clamped gated experts beside a gated
+    shared expert; every norm runs over parts of the row."""
+    z, p = DESIGN_SIZES[size], RIRULIX_SIZES[size]
+    attention = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"],
+                                                "mask": {"size": p["window"], "keep_first": p["keep"]}, "scale": z["dim"] ** -0.5,
+                                                "v_mix": True}}
+    recurrent = {"type": "rglru", "mixer": {"width": z["width"], "blocks": p["blocks"], "conv": p["taps"]}}
+    moe = {"kind": "moe", "router": {"experts": p["experts"], "top": p["top"]}, "expert": {"ff": p["expert_ff"], "limit": 7.0},
+           "shared": {"ff": p["shared_ff"], "limit": 7.0}}
+    return {"architecture": "Rirulix", "torch_dtype": "bfloat16", "width": z["width"], "vocab": DESIGN_VOCAB,
+            "norm": {"eps": 1e-5, "groups": z["groups"]}, "max_positions": CONTEXT,
+            "layers": [dict(recurrent if i % 2 else attention, mlp=moe) for i in range(layers)]}
+
+
 def run_design(args):
     import numpy as np
     import torch
@@ -884,7 +909,8 @@ def run_design(args):
         scratch.cleanup()
         return out
 
-    result = {"design": {"revesun": "Revesun", "pekodra": "Pekodra", "kazodra": "Kazodra", "ladedra": "Ladedra"}[args.design],
+    result = {"design": {"revesun": "Revesun", "pekodra": "Pekodra", "kazodra": "Kazodra", "ladedra": "Ladedra",
+                         "rirulix": "Rirulix"}[args.design],
               "size": args.size,
               "layers": layers,
               "vocab": DESIGN_VOCAB, "dtype": "bf16", "data": "synthetic",
@@ -908,6 +934,17 @@ def run_design(args):
             result["llama"] = measure(llama)
         if args.only in ("all", "kernels"):
             result["kernels"] = ladedra_kernels(args.size, pk)
+        result["clocks"] = sampler.stop(windows)
+        result["peaks"] = pk
+        print(json.dumps(result))
+        return 0
+    if args.design == "rirulix":                   # beside Pekodra: window attention, routed experts, a 32-bit stream
+        if args.only in ("all", "decode", "prefill"):
+            result["rirulix"] = measure(rirulix_config(args.size, layers))
+            result["pekodra"] = measure(pekodra_config(args.size, layers))
+            result["llama"] = measure(llama)
+        if args.only in ("all", "kernels"):
+            result["kernels"] = rirulix_kernels(args.size, pk)
         result["clocks"] = sampler.stop(windows)
         result["peaks"] = pk
         print(json.dumps(result))
@@ -1458,6 +1495,201 @@ def ladedra_kernels(size, pk):
     return out
 
 
+def rirulix_kernels(size, pk):
+    """Rirulix's own kernels alone at this size, timed like :func:`design_kernels`, each behind the like kernel of another
+    model of the package at the same size ("beside: ..."): 2,048 prompt rows of one sequence, and 64 and 8 decoded rows at
+    context 2,048."""
+    import torch
+
+    from tesseract_b200 import kernels
+    from tesseract_b200.parts import Runtime
+    from tesseract_b200.parts.linear import Linear
+
+    z, p = DESIGN_SIZES[size], RIRULIX_SIZES[size]
+    dev, bf16 = "cuda", torch.bfloat16
+    W, page, parts = z["width"], PAGE_SIZE, z["groups"]
+    H, G, d = z["heads"], z["kv_heads"], z["dim"]
+    window, keep, blocks, taps = p["window"], p["keep"], p["blocks"], p["taps"]
+    E, top, EF, S = p["experts"], p["top"], p["expert_ff"], W // p["blocks"]
+    channels = (H + 2 * G) * d
+    half_freq = torch.tensor([5e5 ** (-2.0 * i / d) for i in range(d // 2)], dtype=torch.float32, device=dev)
+    bias_weight, bias_rate = torch.rand(H, device=dev) + 0.2, torch.rand(H, device=dev) * 0.3
+    out = {}
+
+    def timed(name, make, nbytes, flops=0, tensor=False):
+        time_launches(pk, out, name, make, nbytes, flops, tensor)
+
+    def rows_of(rows, width, dtype=bf16):
+        return torch.randn(rows, width, device=dev).to(dtype)
+
+    for label, rows, seqs, begin in (("prefill_2048", 2048, 1, 0), ("decode_64", 64, 64, 2047), ("decode_8", 8, 8, 2047)):
+        new = rows // seqs
+        positions = (torch.arange(rows, dtype=torch.int32, device=dev) % new) + begin
+        seq_of_row = torch.arange(rows, dtype=torch.int32, device=dev) // new
+        row_start = torch.arange(seqs + 1, dtype=torch.int32, device=dev) * new
+        seq_begin = torch.full((seqs,), begin, dtype=torch.int32, device=dev)
+        slots = torch.arange(seqs, dtype=torch.int32, device=dev)
+        pages_per_seq = 2048 // page
+        table = (torch.arange(seqs * pages_per_seq, dtype=torch.int32, device=dev) + 1).view(seqs, pages_per_seq)
+        page_elems = G * page * 2 * d
+        new_pages = lambda: torch.randn(seqs * pages_per_seq + 1, page_elems, device=dev).to(bf16)
+
+        def norms(kind, count):
+            def make(k):
+                res, upd = rows_of(rows, W, torch.float32), rows_of(rows, W, torch.float32)
+                w, b = torch.ones(W, device=dev), torch.zeros(W, device=dev)
+                y = torch.empty(rows, W, dtype=bf16, device=dev)
+                norm = (kind, w, b if kind == kernels.NORM_LAYER else None, count)
+                return lambda: kernels.norm_add_norm(res, upd, norm, norm, y, None, 1e-5)
+            return make
+
+        timed(f"norm_add_norm (RMS over parts)/{label}", norms(kernels.NORM_RMS, parts), rows * W * (4 * 3 + 2))
+        timed(f"beside: norm_add_norm (layer norms, Kazodra)/{label}", norms(kernels.NORM_LAYER, 1), rows * W * (4 * 3 + 2))
+
+        def embed(k):
+            tokens = torch.randint(0, DESIGN_VOCAB, (rows,), dtype=torch.int32, device=dev)
+            tab, pos = rows_of(DESIGN_VOCAB, W), rows_of(2048, W)
+            w, y = torch.ones(W, device=dev), torch.empty(rows, W, device=dev)
+            return lambda: kernels.embedding_norm(tokens, positions, tab, pos, w, parts, 1e-5, y)
+
+        timed(f"embedding_norm/{label}", embed, rows * W * (2 + 2 + 4))
+
+        def bias_cache(k):
+            proj, q, cache = rows_of(rows, channels), torch.empty(rows, H * d, dtype=bf16, device=dev), new_pages()
+            bias, first, mix = torch.randn(channels, device=dev), torch.randn(rows, G * d, device=dev), torch.full((1,), 0.3, device=dev)
+            return lambda: kernels.rope_norm_cache(proj, q, cache, positions, seq_of_row, table, None, amplitude=1.0, heads=H,
+                                                   kv_heads=G, dim=d, vdim=d, rot_dims=0, unit_norm=False, eps=0.0,
+                                                   page_size=page, bias=bias, mix_values=(first, mix))
+
+        timed(f"rope_norm_cache (biases, mixed values)/{label}", bias_cache, rows * (channels * 4 + G * d * 4))
+
+        def rotate(k):
+            proj, q, cache = rows_of(rows, channels), torch.empty(rows, H * d, dtype=bf16, device=dev), new_pages()
+            return lambda: kernels.rope_norm_cache(proj, q, cache, positions, seq_of_row, table, half_freq, amplitude=1.0,
+                                                   heads=H, kv_heads=G, dim=d, vdim=d, rot_dims=d, unit_norm=True, eps=1e-5,
+                                                   page_size=page)
+
+        timed(f"beside: rope_norm_cache (rotation, unit norm, Pekodra)/{label}", rotate, rows * channels * 4)
+
+        def attend(kernel, extras):
+            def make(k):
+                q, y, cache = rows_of(rows, H * d), torch.empty(rows, H * d, dtype=bf16, device=dev), new_pages()
+                common = dict(heads=H, kv_heads=G, dim=d, vdim=d, page_size=page, mask_kind=kernels.MASK_WINDOW, mask_size=window,
+                              scale=d ** -0.5, **extras)
+                if kernel == "prompt":
+                    return lambda: kernels.attention_prompt_mma(q, y, cache, positions, row_start, table, num_seqs=seqs, **common)
+                if kernel == "rows":
+                    return lambda: kernels.attention_rows_mma(q, y, cache, positions, seq_of_row, table, **common)
+                return lambda: kernels.attention_masked(q, None, y, cache, positions, seq_of_row, table, sink=False, **common)
+            return make
+
+        seen = sum(min(window, int(t) + 1) + min(keep, max(0, int(t) + 1 - window)) for t in positions.tolist())
+        moved = rows * H * d * 2 * 2 + (seqs * min(begin + new, window + keep) if new == 1 else rows) * 2 * G * d * 2
+        flops = seen * H * d * 4
+        kind = "prompt" if rows > 256 else "rows"
+        own = {"keep_first": keep, "distance_bias": (bias_weight, bias_rate)}
+        timed(f"attention_{kind}_mma (window {window}, {keep} kept, distance bias)/{label}", attend(kind, own), moved, flops, True)
+        timed(f"beside: attention_{kind}_mma (window {window}, Pekodra)/{label}", attend(kind, {}), moved, flops, True)
+        timed(f"attention_masked (window {window}, {keep} kept, distance bias)/{label}", attend("masked", own), moved, flops)
+        timed(f"beside: attention_masked (window {window})/{label}", attend("masked", {}), moved, flops)
+
+        def conv(k):
+            proj, u = rows_of(rows, 2 * W), torch.empty(rows, W, dtype=bf16, device=dev)
+            w, bx, bc = torch.randn(taps, W, device=dev), torch.randn(W, device=dev), torch.randn(W, device=dev)
+            state = torch.zeros(seqs + 1, taps - 1, W, device=dev)
+            return lambda: kernels.short_conv(proj[:, W:], bx, w, bc, state, u, positions, seq_of_row, row_start, seq_begin, slots,
+                                              num_seqs=seqs, single=new == 1)
+
+        timed(f"short_conv (with its state)/{label}", conv, rows * W * 4 + seqs * (taps - 1) * W * (8 if new == 1 else 4))
+
+        def gates_of(k):
+            u, gates = rows_of(rows, W), rows_of(blocks * 2 * S, S).view(blocks, 2 * S, S)
+            return u, gates, torch.randn(W, device=dev), torch.randn(W, device=dev), -torch.rand(W, device=dev)
+
+        if new == 1:
+            def step(k):
+                u, gates, br, bi, rate = gates_of(k)
+                y, by, o = rows_of(rows, 2 * W), torch.randn(W, device=dev), torch.empty(rows, W, dtype=bf16, device=dev)
+                state = torch.zeros(seqs + 1, W, device=dev)
+                return lambda: kernels.rglru_step(u, gates, br, bi, rate, y[:, :W], by, state, slots, o)
+
+            timed(f"rglru_step (gates, recurrence, output gate)/{label}", step, rows * W * (2 + 2 + 2 + 8) + 2 * W * S * 2,
+                  flops=rows * W * S * 4, tensor=True)
+        else:
+            def gates(k):
+                u, gates, br, bi, rate = gates_of(k)
+                pairs = torch.empty(rows, W, 2, device=dev)
+                return lambda: kernels.rglru_gates(u, gates, br, bi, rate, pairs)
+
+            timed(f"rglru_gates/{label}", gates, rows * W * (2 + 8) + 2 * W * S * 2, flops=rows * W * S * 4, tensor=True)
+
+            def scan(k):
+                pairs, y, by = torch.rand(rows, W, 2, device=dev) * 0.5, rows_of(rows, 2 * W), torch.randn(W, device=dev)
+                o, state = torch.empty(rows, W, dtype=bf16, device=dev), torch.zeros(seqs + 1, W, device=dev)
+                return lambda: kernels.rglru_scan(pairs, y[:, :W], by, state, o, row_start, slots, num_seqs=seqs, max_new=new)
+
+            timed(f"rglru_scan/{label}", scan, rows * W * (8 + 2 + 2))
+
+        def mingru(k):
+            proj, o = rows_of(rows, 3 * W, torch.float32), torch.empty(rows, W, dtype=bf16, device=dev)
+            bz, bx, state = torch.randn(W, device=dev), torch.randn(W, device=dev), torch.zeros(seqs + 1, W, device=dev)
+            return lambda: kernels.gated_recurrence(proj, bz, bx, state, o, row_start, slots, num_seqs=seqs, max_new=new)
+
+        timed(f"beside: gated_recurrence (minGRU, Revesun)/{label}", mingru, rows * W * (12 + 2) + (seqs * W * 8 if new == 1 else 0))
+
+        def route(k):
+            x = rows_of(rows, W)
+            router = Linear(torch.randn(-(-(E + 1) // 16) * 16, W).to(bf16), Runtime(bf16, torch.device(dev)))
+            ids = torch.empty(rows, top, dtype=torch.int32, device=dev)
+            weights = torch.empty(rows, top, dtype=torch.float32, device=dev)
+            return lambda: kernels.choose_sigmoid(router.forward(x, float32_out=True), E, ids, weights)
+
+        timed(f"router (product with 32-bit logits, choice)/{label}", route, rows * W * 2 + E * W * 2, flops=rows * E * W * 2)
+
+        ids = torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(rows)]).to(torch.int32).contiguous()
+        offsets = torch.empty(E + 1, dtype=torch.int32, device=dev)
+        order = torch.empty(rows * top, dtype=torch.int32, device=dev)
+        kernels.expert_plan(ids, E, offsets, order)
+        used = min(E, rows * top)                      # experts whose weights a step must read
+
+        def experts_up(fused):
+            def make(k):
+                x, up = rows_of(rows, W), torch.randn(E, 2 * EF, W, device=dev).to(bf16)
+                weights = torch.rand(rows * top, device=dev)
+                hidden = torch.empty(rows * top, EF if fused else 2 * EF, dtype=bf16, device=dev)
+                if fused:
+                    return lambda: kernels.expert_linear(x, up, hidden, offsets, order, source_div=top, row_weights=weights,
+                                                         epilogue=kernels.EXPERT_GATED_CLAMPED, limit=7.0, slope=1.702)
+                return lambda: kernels.expert_linear(x, up, hidden, offsets, order, source_div=top)
+            return make
+
+        weight_bytes = used * 2 * EF * W * 2 + rows * W * 2
+        timed(f"expert_linear gate and up, weighed and gated/{label}", experts_up(True), weight_bytes + rows * top * EF * 2,
+              flops=rows * top * 2 * EF * W * 2, tensor=True)
+        timed(f"beside: expert_linear gate and up, plain (Ladedra)/{label}", experts_up(False), weight_bytes + rows * top * 2 * EF * 2,
+              flops=rows * top * 2 * EF * W * 2, tensor=True)
+
+        def combine(own):
+            def make(k):
+                y, base, gate = rows_of(rows * top, W, torch.float32), rows_of(rows, W, torch.float32), torch.randn(rows, 48, device=dev)
+                weights = None if own else torch.rand(rows, top, device=dev)
+                return lambda: kernels.expert_combine(y, weights, base, base, base_gate=gate[:, E] if own else None)
+            return make
+
+        timed(f"expert_combine (gated base)/{label}", combine(True), rows * W * 4 * (top + 2))
+        timed(f"beside: expert_combine (weights, Pekodra)/{label}", combine(False), rows * W * 4 * (top + 2))
+
+        def shared_gate(activation):
+            def make(k):
+                gu, y = rows_of(rows, 2 * p["shared_ff"]), torch.empty(rows, p["shared_ff"], dtype=bf16, device=dev)
+                return lambda: kernels.gated_activation(gu, None, y, activation, limit=7.0, slope=1.702)
+            return make
+
+        timed(f"gated_activation (clamped)/{label}", shared_gate(kernels.ACT_CLAMPED), rows * p["shared_ff"] * 2 * 3)
+        timed(f"beside: gated_activation (SiLU, Ladedra)/{label}", shared_gate(kernels.ACT_SILU), rows * p["shared_ff"] * 2 * 3)
+    return out
+
+
 def pekodra_kernels(size, pk):
     """Pekodra's own kernels alone at this size, timed like :func:`design_kernels`: 2,048 prompt rows of one sequence,
     and 64 decoded rows at context 2,048."""
@@ -1660,7 +1892,7 @@ def main():
     parser.add_argument("--workload", choices=["3b", "8b"], default=None,
                         help="run another workload instead of the headline one: continuous batching at the 3B sizes, "
                              "or a 2,048-token portion beside 64 decode rows at the 8B sizes")
-    parser.add_argument("--design", choices=["revesun", "pekodra", "kazodra", "ladedra"], default=None,
+    parser.add_argument("--design", choices=["revesun", "pekodra", "kazodra", "ladedra", "rirulix"], default=None,
                         help="instead of the headline workload: prefill and decode of this design beside a Llama of "
                              "equal layer sizes (--size), and the design's own kernels alone")
     args = parser.parse_args()

@@ -170,8 +170,13 @@ class RoutedExperts(FeedForward):
         if isinstance(x, DeferredNorm):
             x = x.materialize()
         rows, device = x.shape[0], x.device
-        logits = self.router.forward(x, float32_out=True)
-        ids, weights = self.choose(logits)
+        base_gate = None
+        if self.gated_shared:
+            logits = self.router.forward(x, float32_out=True)
+            base_gate = logits[:, self.num_experts]             # the shared expert's own logit
+            ids, weights = self.choose(logits)
+        else:
+            ids, weights = self.route(x)
         count = rows * self.top_k
         offsets = torch.empty(self.num_experts + 1, dtype=torch.int32, device=device)
         order = torch.empty(count, dtype=torch.int32, device=device)
@@ -205,8 +210,7 @@ class RoutedExperts(FeedForward):
                 kernels.squared_relu(z, z)
             base = self.shared_down.forward(z, float32_out=True)
         out = base if base is not None else torch.empty((rows, self.hidden_size), dtype=torch.float32, device=device)
-        kernels.expert_combine(parts, None if self.weigh_input else weights, base, out,
-                               base_gate=logits[:, self.num_experts] if self.gated_shared else None)
+        kernels.expert_combine(parts, None if self.weigh_input else weights, base, out, base_gate=base_gate)
         if self.stream_f32 or self.runtime.is_float32:
             return out
         return out.to(self.runtime.dtype)

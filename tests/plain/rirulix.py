@@ -148,13 +148,13 @@ def clamped_expert(w, prefix, h, limit, store=identity):
 
 
 def route(router, logits, gaps=None):
-    """``(chosen experts, weights)`` of one row.  ``gaps`` (a list) receives how far, in scores, the last chosen expert was
+    """``(chosen experts, weights)`` of one row.  ``gaps`` (a list) receives how far, in logits, the last chosen expert was
     from the best one not chosen."""
     scores = sigmoid(logits)
     ranked = sorted(range(router["experts"]), key=lambda e: (-logits[e], e))
     chosen = ranked[:router["top"]]
     if gaps is not None and router["top"] < router["experts"]:
-        gaps.append(scores[chosen[-1]] - scores[ranked[router["top"]]])
+        gaps.append(logits[chosen[-1]] - logits[ranked[router["top"]]])
     return chosen, scores[chosen]
 
 
@@ -167,7 +167,7 @@ def expert_feed_forward(mlp, w, h, store=identity, close_calls=None):
         gaps = []
         chosen, weights = route(mlp["router"], logits[t], gaps)
         if close_calls is not None and gaps:
-            close_calls[t] = min(close_calls.get(t, 1.0), min(gaps))
+            close_calls[t] = min(close_calls.get(t, math.inf), min(gaps))
         for e, weight in zip(chosen, weights):
             out[t] += clamped_expert(w, f"e{e}.", weight * h[t:t + 1], mlp["expert"]["limit"], store)[0]
     if mlp.get("shared"):
