@@ -15,18 +15,35 @@
 //                    run is first reduced to (A, B) with S_end = A S_start + B, the runs are chained from the slot's state,
 //                    and every run is walked again from its own start.
 //
-// 1 - a^2 is taken as -expm1(2 log a): a is close to 1 where the unit remembers.  Everything behind the two products'
+// 1 - a^2 is taken as -(e^(2 log a) - 1) by that function's series where a is close to 1, as it is where the unit remembers.
+// a itself takes the accurate exponential: its error is multiplied once a token for as long as a channel remembers; the
+// sigmoids' and the output's divisions are single hardware approximations (an ulp or two).  Everything behind the two products'
 // 32-bit sums is 32-bit; products of bfloat16 operands are exact in those sums.
 #include "common.cuh"
 
 namespace {
 
-__device__ __forceinline__ float sigmoid_f32(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f32(float x) { return __fdividef(1.0f, 1.0f + expf(-x)); }
+// 0.5 z (1 + tanh(k (z + 0.044715 z^3))) = z sigmoid(2 k (z + 0.044715 z^3)), k = sqrt(2 / pi)
 __device__ __forceinline__ float gelu_tanh_f32(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    return z * sigmoid_f32(1.5957691216057308f * (z + 0.044715f * z * z * z));
+}
+// sqrt(1 - a^2) from log a <= 0 and a = e^(log a)
+__device__ __forceinline__ float entering(float log_a, float a) {
+    const float z = 2.0f * log_a;
+    // 1 - e^z = -z (1 + z/2 (1 + z/3 (1 + ...))): eight terms, good to 1e-8 for |z| <= 1/2
+    float series = fmaf(z, 1.0f / 8.0f, 1.0f);
+    series = fmaf(z * (1.0f / 7.0f), series, 1.0f);
+    series = fmaf(z * (1.0f / 6.0f), series, 1.0f);
+    series = fmaf(z * (1.0f / 5.0f), series, 1.0f);
+    series = fmaf(z * (1.0f / 4.0f), series, 1.0f);
+    series = fmaf(z * (1.0f / 3.0f), series, 1.0f);
+    series = fmaf(z * 0.5f, series, 1.0f);
+    return sqrtf(z > -0.5f ? -z * series : fmaf(-a, a, 1.0f));
 }
 
-// What stands behind the gates' product, per (row, channel).
+// What stands behind the gates' product, per (row, channel).  A thread first asks for all it reads of a row's channels
+// (load), then finishes one after the other: what it stores never hides what it has yet to read.
 template <typename T>
 struct Behind {
     const T* u;                   // [rows, width]
@@ -42,19 +59,35 @@ struct Behind {
     int64_t out_stride;
     int width;
 
-    __device__ __forceinline__ void operator()(int row, int c, float acc_r, float acc_i) const {
-        const float r = sigmoid_f32(acc_r + bias_r[c]), i = sigmoid_f32(acc_i + bias_i[c]);
-        const float log_a = rate[c] * r;
+    struct Taken {
+        float u, br, bi, rate, state, y;
+    };
+    __device__ __forceinline__ int64_t state_row(int row) const { return pairs == nullptr ? (int64_t)slots[row] * width : 0; }
+    __device__ __forceinline__ Taken load(int row, int64_t at_state, int c) const {
+        Taken t;
+        t.u = Elem<T>::load(u + (int64_t)row * u_stride + c);
+        t.br = bias_r[c];
+        t.bi = bias_i[c];
+        t.rate = rate[c];
+        t.state = t.y = 0.0f;
+        if (pairs == nullptr) {
+            t.state = state[at_state + c];
+            t.y = Elem<T>::load(y + (int64_t)row * y_stride + c) + y_bias[c];
+        }
+        return t;
+    }
+    __device__ __forceinline__ void finish(int row, int64_t at_state, int c, float acc_r, float acc_i, const Taken& t) const {
+        const float r = sigmoid_f32(acc_r + t.br), i = sigmoid_f32(acc_i + t.bi);
+        const float log_a = t.rate * r;
         const float a = expf(log_a);
-        const float x = sqrtf(-expm1f(2.0f * log_a)) * i * Elem<T>::load(u + (int64_t)row * u_stride + c);
+        const float x = entering(log_a, a) * i * t.u;
         if (pairs != nullptr) {
             pairs[(int64_t)row * width + c] = make_float2(a, x);
             return;
         }
-        float* at = state + (int64_t)slots[row] * width + c;
-        const float s = fmaf(a, *at, x);
-        *at = s;
-        Elem<T>::store(out + (int64_t)row * out_stride + c, s * gelu_tanh_f32(Elem<T>::load(y + (int64_t)row * y_stride + c) + y_bias[c]));
+        const float s = fmaf(a, t.state, x);
+        state[at_state + c] = s;
+        Elem<T>::store(out + (int64_t)row * out_stride + c, s * gelu_tanh_f32(t.y));
     }
 };
 
@@ -112,19 +145,20 @@ rglru_gates_kernel(const T* __restrict__ W, Behind<T> behind, int rows, int S) {
     for (int i = 0; i < 4; ++i) {
         const int row = r0 + ty * 4 + i;
         if (row >= rows) continue;
+        const int64_t at_state = behind.state_row(row);
 #pragma unroll
         for (int j = 0; j < 4; j += 2) {
-            const int n = n0 + tx * 4 + j;                       // even: r of channel n / 2, and i beside it
-            if (n < N) behind(row, b * S + n / 2, acc[i][j], acc[i][j + 1]);
+            const int n = n0 + tx * 4 + j, c = b * S + n / 2;    // n even: r of channel n / 2, and i beside it
+            if (n < N) behind.finish(row, at_state, c, acc[i][j], acc[i][j + 1], behind.load(row, at_state, c));
         }
     }
 }
 
-// bfloat16 on the tensor cores (mma.sync m16n8k16, 32-bit accumulators), S a multiple of 64: eight warps take 64 rows by 128
-// output rows (64 channels) of one block, a warp 32 by 32; K in steps of 64 through a ring of three stages that cp.async
-// fills two steps ahead, 16-byte chunks of a row XOR-swizzled by the row.
-constexpr int PM = 64, PN = 128, PK = 64, PSTAGES = 3;
-constexpr int kPipeSmem = PSTAGES * (PM + PN) * PK * 2;
+// bfloat16 on the tensor cores (mma.sync m16n8k16, 32-bit accumulators), S a multiple of 64: WM x WN warps of 16 MI rows by
+// 16 NJ output rows each; K in steps of 64 through a ring of three stages that cp.async fills two steps ahead, 16-byte
+// chunks of a row XOR-swizzled by the row.  Two shapes: 64 rows by 128 output rows (64 channels) of a block for prompt
+// portions, 16 by 64 in steps of few rows.
+constexpr int PK = 64, PSTAGES = 3;
 
 __device__ __forceinline__ void mma_bf16_16816(float* c, const uint32_t* a, const uint32_t* b) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -144,46 +178,45 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t* r, uint32_t addr) {
 // byte offset of 16-byte chunk `chunk` (0..7) of row `row` in a tile whose rows are 128 bytes
 __device__ __forceinline__ uint32_t swizzled(int row, int chunk) { return (uint32_t)(row * 128 + ((chunk ^ (row & 7)) << 4)); }
 
-__global__ void __launch_bounds__(256)
+template <int MI, int NJ, int WM, int WN>
+struct Shape {
+    static constexpr int PM = 16 * MI * WM, PN = 16 * NJ * WN, THREADS = 32 * WM * WN;
+    static constexpr int STAGE = (PM + PN) * 128, SMEM = PSTAGES * STAGE;
+    static constexpr int A_CHUNKS = PM * 8 / THREADS, W_CHUNKS = PN * 8 / THREADS;
+    static_assert(PM * 8 % THREADS == 0 && PN * 8 % THREADS == 0, "every thread copies as many chunks");
+};
+
+template <int MI, int NJ, int WM, int WN>
+__global__ void __launch_bounds__(32 * WM * WN)
 rglru_gates_mma_kernel(const __nv_bfloat16* __restrict__ W, Behind<__nv_bfloat16> behind, int rows, int S) {
+    using Sh = Shape<MI, NJ, WM, WN>;
     extern __shared__ __align__(128) unsigned char pipe_smem[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int N = 2 * S, b = blockIdx.z, n0 = blockIdx.x * PN, r0 = blockIdx.y * PM;
+    const int N = 2 * S, b = blockIdx.z, n0 = blockIdx.x * Sh::PN, r0 = blockIdx.y * Sh::PM;
     const __nv_bfloat16* Wb = W + (int64_t)b * N * S;
     const uint32_t base = (uint32_t)__cvta_generic_to_shared(pipe_smem);
-    // what this thread copies every step: two chunks of A (64 rows x 8 chunks) and four of W (128 rows x 8 chunks)
-    const __nv_bfloat16* a_src[2];
-    uint32_t a_dst[2];
-    int a_bytes[2];
-#pragma unroll
-    for (int p = 0; p < 2; ++p) {
-        const int c = tid + p * 256, r = c >> 3, chunk = c & 7;
-        const bool there = r0 + r < rows;
-        a_bytes[p] = there ? 16 : 0;
-        a_src[p] = behind.u + (there ? (int64_t)(r0 + r) * behind.u_stride : 0) + (int64_t)b * S + chunk * 8;
-        a_dst[p] = swizzled(r, chunk);
-    }
-    const __nv_bfloat16* w_src[4];
-    uint32_t w_dst[4];
-    int w_bytes[4];
-#pragma unroll
-    for (int p = 0; p < 4; ++p) {
-        const int c = tid + p * 256, r = c >> 3, chunk = c & 7;
-        const int n = n0 + r;
-        w_bytes[p] = n < N ? 16 : 0;
-        w_src[p] = Wb + (n < N ? (int64_t)n * S : 0) + chunk * 8;
-        w_dst[p] = PM * 128 + swizzled(r, chunk);
-    }
+    // a thread's chunks: chunk `tid & 7` of rows tid / 8, tid / 8 + THREADS / 8, ... of A and of W
+    const int copy_row = tid >> 3, chunk = tid & 7;
+    constexpr int ROW_STEP = Sh::THREADS / 8;
     const int steps = S / PK;
     auto fill_w = [&](int step) {
-        const uint32_t stage = base + (uint32_t)(step % PSTAGES) * (PM + PN) * 128;
+        const uint32_t stage = base + (uint32_t)(step % PSTAGES) * Sh::STAGE + Sh::PM * 128;
 #pragma unroll
-        for (int p = 0; p < 4; ++p) cp_async16(stage + w_dst[p], w_src[p] + step * PK, w_bytes[p]);
+        for (int p = 0; p < Sh::W_CHUNKS; ++p) {
+            const int r = copy_row + p * ROW_STEP, n = n0 + r;
+            cp_async16(stage + swizzled(r, chunk), Wb + (n < N ? (int64_t)n * S : 0) + chunk * 8 + step * PK, n < N ? 16 : 0);
+        }
     };
     auto fill_a = [&](int step) {
-        const uint32_t stage = base + (uint32_t)(step % PSTAGES) * (PM + PN) * 128;
+        const uint32_t stage = base + (uint32_t)(step % PSTAGES) * Sh::STAGE;
 #pragma unroll
-        for (int p = 0; p < 2; ++p) cp_async16(stage + a_dst[p], a_src[p] + step * PK, a_bytes[p]);
+        for (int p = 0; p < Sh::A_CHUNKS; ++p) {
+            const int r = copy_row + p * ROW_STEP;
+            const bool there = r0 + r < rows;
+            cp_async16(stage + swizzled(r, chunk),
+                       behind.u + (there ? (int64_t)(r0 + r) * behind.u_stride : 0) + (int64_t)b * S + chunk * 8 + step * PK,
+                       there ? 16 : 0);
+        }
     };
     pdl_trigger();
     for (int s = 0; s < PSTAGES - 1; ++s)              // weights do not depend on the kernel in front
@@ -193,12 +226,12 @@ rglru_gates_mma_kernel(const __nv_bfloat16* __restrict__ W, Behind<__nv_bfloat16
         if (s < steps) fill_a(s);
         cp_async_commit();                             // (the first group also holds the weights of both stages)
     }
-    const int wm = warp >> 2, wn = warp & 3;           // the warp's 32 x 32 part of the tile
-    float acc[2][4][4];
+    const int wm = warp / WN, wn = warp % WN;          // the warp's part of the tile
+    float acc[MI][2 * NJ][4];
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
+    for (int i = 0; i < MI; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+        for (int j = 0; j < 2 * NJ; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.0f;
     for (int step = 0; step < steps; ++step) {
@@ -209,38 +242,60 @@ rglru_gates_mma_kernel(const __nv_bfloat16* __restrict__ W, Behind<__nv_bfloat16
             fill_a(step + PSTAGES - 1);
         }
         cp_async_commit();
-        const uint32_t stage = base + (uint32_t)(step % PSTAGES) * (PM + PN) * 128;
+        const uint32_t stage = base + (uint32_t)(step % PSTAGES) * Sh::STAGE;
 #pragma unroll
         for (int ks = 0; ks < PK / 16; ++ks) {
-            uint32_t a[2][4], bb[2][4];
+            uint32_t a[MI][4], bb[NJ][4];
 #pragma unroll
-            for (int i = 0; i < 2; ++i)
-                ldmatrix_x4(a[i], stage + swizzled(wm * 32 + i * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+            for (int i = 0; i < MI; ++i)
+                ldmatrix_x4(a[i], stage + swizzled((wm * MI + i) * 16 + (lane & 15), ks * 2 + (lane >> 4)));
 #pragma unroll
-            for (int j = 0; j < 2; ++j)                // two n-tiles of eight output rows a load
-                ldmatrix_x4(bb[j], stage + PM * 128 +
-                                       swizzled(wn * 32 + j * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1)));
+            for (int j = 0; j < NJ; ++j)               // two n-tiles of eight output rows a load
+                ldmatrix_x4(bb[j], stage + Sh::PM * 128 +
+                                       swizzled((wn * NJ + j) * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1)));
 #pragma unroll
-            for (int i = 0; i < 2; ++i)
+            for (int i = 0; i < MI; ++i)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) mma_bf16_16816(acc[i][j], a[i], &bb[j >> 1][(j & 1) * 2]);
+                for (int j = 0; j < 2 * NJ; ++j) mma_bf16_16816(acc[i][j], a[i], &bb[j >> 1][(j & 1) * 2]);
         }
     }
     cp_async_wait<0>();
     const int g = lane >> 2, t = lane & 3;
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
+    for (int i = 0; i < MI; ++i)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-            const int row = r0 + wm * 32 + i * 16 + g + half * 8;
+            const int row = r0 + (wm * MI + i) * 16 + g + half * 8;
             if (row >= rows) continue;
+            const int64_t at_state = behind.state_row(row);
+            typename Behind<__nv_bfloat16>::Taken taken[2 * NJ];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const int n = n0 + wn * 32 + j * 8 + 2 * t;      // even: r of channel n / 2, and i beside it
-                if (n < N) behind(row, b * S + n / 2, acc[i][j][half * 2], acc[i][j][half * 2 + 1]);
+            for (int j = 0; j < 2 * NJ; ++j) {         // n even: r of channel n / 2, and i beside it
+                const int n = n0 + (wn * 2 * NJ + j) * 8 + 2 * t;
+                if (n < N) taken[j] = behind.load(row, at_state, b * S + n / 2);
+            }
+#pragma unroll
+            for (int j = 0; j < 2 * NJ; ++j) {
+                const int n = n0 + (wn * 2 * NJ + j) * 8 + 2 * t;
+                if (n < N) behind.finish(row, at_state, b * S + n / 2, acc[i][j][half * 2], acc[i][j][half * 2 + 1], taken[j]);
             }
         }
 }
+
+template <int MI, int NJ, int WM, int WN>
+int launch_gates_mma(const __nv_bfloat16* W, const Behind<__nv_bfloat16>& behind, int rows, int blocks, int S, cudaStream_t stream) {
+    using Sh = Shape<MI, NJ, WM, WN>;
+    auto kernel = rglru_gates_mma_kernel<MI, NJ, WM, WN>;
+    const dim3 grid((2 * S + Sh::PN - 1) / Sh::PN, (rows + Sh::PM - 1) / Sh::PM, blocks);
+    if (grid.y > 65535) return TB_ERR_BAD_SIZE;
+    if (Sh::SMEM > 40 * 1024) {
+        cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Sh::SMEM);
+        if (err != cudaSuccess) return (int)err;
+    }
+    cudaError_t launched = tb_launch_pdl(kernel, grid, dim3(Sh::THREADS), (size_t)Sh::SMEM, stream, W, behind, rows, S);
+    return launched == cudaSuccess ? tb_launch_status() : (int)launched;
+}
+constexpr int kFewRows = 256;       // up to here a step takes the small tiles (a choice by the row count alone)
 
 constexpr int kChannels = 16;       // channels of a block that cuts its rows into runs
 constexpr int kMaxRuns = 64;        // runs of rows of a block (threads = runs * channels)
@@ -320,13 +375,10 @@ TB_EXPORT int tb_rglru_gates(const void* u, int64_t u_stride, const void* W, con
     const int width = blocks * S;
     cudaError_t launched;
     if (dtype == TB_BF16 && S % PK == 0 && u_stride % 8 == 0 && ((uintptr_t)u | (uintptr_t)W) % 16 == 0) {
-        const dim3 grid((2 * S + PN - 1) / PN, (rows + PM - 1) / PM, blocks);
-        cudaError_t err = cudaFuncSetAttribute(rglru_gates_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kPipeSmem);
-        if (err != cudaSuccess) return (int)err;
-        launched = tb_launch_pdl(rglru_gates_mma_kernel, grid, dim3(256), (size_t)kPipeSmem, stream, (const __nv_bfloat16*)W,
-                                 behind_of<__nv_bfloat16>(u, u_stride, bias_r, bias_i, rate, pairs, state, state_slots, y,
-                                                          y_stride, y_bias, out, out_stride, width), rows, S);
-        return launched == cudaSuccess ? tb_launch_status() : (int)launched;
+        const auto behind = behind_of<__nv_bfloat16>(u, u_stride, bias_r, bias_i, rate, pairs, state, state_slots, y, y_stride,
+                                                     y_bias, out, out_stride, width);
+        return rows <= kFewRows ? launch_gates_mma<1, 1, 1, 4>((const __nv_bfloat16*)W, behind, rows, blocks, S, stream)
+                                : launch_gates_mma<2, 2, 2, 4>((const __nv_bfloat16*)W, behind, rows, blocks, S, stream);
     }
     const dim3 grid((2 * S + BN - 1) / BN, (rows + BM - 1) / BM, blocks);
     if (dtype == TB_F32)

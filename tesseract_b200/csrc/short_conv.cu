@@ -62,7 +62,7 @@ __device__ __forceinline__ void store_floats(float* p, const float* v) {
 }
 
 // A thread a packet of channels for kRowTile neighbouring rows in turn: rows of one sequence slide through the
-// registers, so every projected packet is read once (and J - 1 times more where a tile begins).
+// registers, so every projected packet is read once (and the J - 1 packets in front of a tile once more).
 constexpr int kRowTile = 8;
 
 template <typename T, bool SINGLE, int J>
@@ -86,36 +86,51 @@ short_conv_packets_kernel(const T* __restrict__ proj, int64_t proj_stride, const
     if (in_bias != nullptr) load_floats<N>(in_bias + c0, add);
     if (out_bias != nullptr) load_floats<N>(out_bias + c0, behind);
     pdl_wait();                                   // (weights above; the projected rows come from the kernel in front)
+    // the tile's own rows and their sequences, asked for at once
+    uint4 own[ROWS];
+    int row_seq[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const int row = min(blockIdx.x * ROWS + r, rows - 1);
+        own[r] = *reinterpret_cast<const uint4*>(proj + (int64_t)row * proj_stride + c0);
+        row_seq[r] = seq_of_row[row];
+    }
     float v[J][N];
     int seq_before = -1;
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
         const int row = blockIdx.x * ROWS + r;
         if (row >= rows) return;
-        const int seq = seq_of_row[row], pos = positions[row];
-        const int begin = seq_begin[seq], first_row = row_start[seq];
+        const int seq = row_seq[r];
         const bool slides = r > 0 && seq == seq_before;       // the row in front is the position in front
         seq_before = seq;
-        float* st = state + (int64_t)state_slots[seq] * (J - 1) * channels + c0;
+        float* st = nullptr;
+        if (slides) {
 #pragma unroll
-        for (int j = 0; j < J; ++j) {
-            if (slides && j < J - 1) {
+            for (int j = 0; j + 1 < J; ++j)
 #pragma unroll
                 for (int e = 0; e < N; ++e) v[j][e] = v[j + 1][e];
-                continue;
-            }
-            const int p = pos - (J - 1) + j;
-            if (p >= begin) {
-                Packet<T>::load(proj + (int64_t)(first_row + (p - begin)) * proj_stride + c0, v[j]);
+        } else {
+            const int pos = positions[row], begin = seq_begin[seq], first_row = row_start[seq];
+            st = state + (int64_t)state_slots[seq] * (J - 1) * channels + c0;
 #pragma unroll
-                for (int e = 0; e < N; ++e) v[j][e] += add[e];
-            } else if (p >= 0) {
-                load_floats<N>(st + (int64_t)(p - (begin - (J - 1))) * channels, v[j]);
-            } else {
+            for (int j = 0; j + 1 < J; ++j) {
+                const int p = pos - (J - 1) + j;
+                if (p >= begin) {
+                    Packet<T>::load(proj + (int64_t)(first_row + (p - begin)) * proj_stride + c0, v[j]);
 #pragma unroll
-                for (int e = 0; e < N; ++e) v[j][e] = 0.0f;
+                    for (int e = 0; e < N; ++e) v[j][e] += add[e];
+                } else if (p >= 0) {
+                    load_floats<N>(st + (int64_t)(p - (begin - (J - 1))) * channels, v[j]);
+                } else {
+#pragma unroll
+                    for (int e = 0; e < N; ++e) v[j][e] = 0.0f;
+                }
             }
         }
+        Packet<T>::unpack(own[r], v[J - 1]);
+#pragma unroll
+        for (int e = 0; e < N; ++e) v[J - 1][e] += add[e];
         float y[N];
 #pragma unroll
         for (int e = 0; e < N; ++e) {
