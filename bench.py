@@ -1650,7 +1650,7 @@ def rirulix_kernels(size, pk):
         offsets = torch.empty(E + 1, dtype=torch.int32, device=dev)
         order = torch.empty(rows * top, dtype=torch.int32, device=dev)
         kernels.expert_plan(ids, E, offsets, order)
-        used = min(E, rows * top)                      # experts whose weights a step must read
+        used = int(ids.unique().numel())               # experts whose weights a step must read
 
         def experts_up(fused):
             def make(k):

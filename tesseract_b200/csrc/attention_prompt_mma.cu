@@ -342,7 +342,7 @@ attention_prompt_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __re
 // are the 16 rows of the first operand, so a key or value is fetched once for all of them; the block's four warps
 // share every tile of 64 keys, 16 keys a warp, each with a streaming softmax of its own, and their partial results
 // (maximum, sum, accumulator) meet in shared memory in warp order.
-template <int D, int DV>
+template <int D, int DV, bool BIASED>
 __global__ void __launch_bounds__(128)
 attention_rows_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__ out, int64_t out_stride,
                       const bf16* __restrict__ cache, const int* __restrict__ positions,
@@ -421,9 +421,8 @@ attention_rows_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __rest
                 l[r] = t == 0 ? 1.0f : 0.0f;
             }
     }
-    const bool biased = x.bias_weight != nullptr;
     float bias_weight[2] = {0.0f, 0.0f}, bias_rate[2] = {0.0f, 0.0f};
-    if (biased) {
+    if (BIASED) {
 #pragma unroll
         for (int r = 0; r < 2; ++r)
             if (g + r * 8 < per) {
@@ -467,7 +466,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __rest
                 for (int e = 0; e < 4; ++e) {
                     const int at = at0 + j * 8 + 2 * t + (e & 1);
                     s[j][e] = at < span ? capped(s[j][e] * scale, x.softcap, x.cap_k) : -1.0e30f;     // (all of the span is inside the mask)
-                    if (biased && at < span) {
+                    if (BIASED && at < span) {
                         const int key = at < blocks ? at : key_lo + at - blocks;
                         s[j][e] -= distance_bias(bias_weight[e >> 1], bias_rate[e >> 1], pos - key);
                     }
@@ -556,7 +555,7 @@ int launch_rows(const void* q, int64_t q_stride, void* out, int64_t out_stride, 
                 int page_size, int mask_kind, int mask_size, float scale, int keys_per_value, int out_f32, Extras x,
                 cudaStream_t stream) {
     constexpr int smem = 2 * KT * (D * 2 + 16 + DV * 2 + 16) + 4 * 16 * (DV + 2) * 4;
-    auto kernel = attention_rows_kernel<D, DV>;
+    auto kernel = x.bias_weight != nullptr ? attention_rows_kernel<D, DV, true> : attention_rows_kernel<D, DV, false>;
     if (smem > 40 * 1024) {
         cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (err != cudaSuccess) return (int)err;
