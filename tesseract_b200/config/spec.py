@@ -65,12 +65,14 @@ class LayerSpec:
     token_input: Optional[PartSpec] = None
     # what weights every sublayer's result on its way into the stream (a block kind that takes one), or None
     residual_gates: Optional[PartSpec] = None
+    # how the copies of a multi-copy stream meet around every sublayer (a block kind that keeps such a stream), or None
+    stream_mixing: Optional[PartSpec] = None
 
     @classmethod
     def make(cls, block: str, mixer: PartSpec, feed_forward: Optional[PartSpec],
              norms: Mapping[str, PartSpec], token_input: Optional[PartSpec] = None,
-             residual_gates: Optional[PartSpec] = None) -> "LayerSpec":
-        return cls(block, mixer, feed_forward, tuple(sorted(norms.items())), token_input, residual_gates)
+             residual_gates: Optional[PartSpec] = None, stream_mixing: Optional[PartSpec] = None) -> "LayerSpec":
+        return cls(block, mixer, feed_forward, tuple(sorted(norms.items())), token_input, residual_gates, stream_mixing)
 
     @property
     def norms(self) -> Dict[str, PartSpec]:

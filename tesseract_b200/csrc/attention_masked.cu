@@ -15,7 +15,8 @@
 //   sink     the softmax denominator has one more entry that carries no value, of score 0
 //            (w_j = exp(s_j) / (1 + sum_j exp(s_j))) or, with `sinks`, of a learned score per query head;
 //   softcap  with softcap > 0 a score s becomes softcap * tanh(s / softcap) (the sink's score is not touched);
-//   gate     the output is multiplied, element by element, by sigmoid(gate[row, head, :]).
+//   gate     the output is multiplied, element by element, by sigmoid(gate[row, head, :]), or, with `head_gate`, as a whole
+//            by the sigmoid of one number per row and head.
 //
 // One warp per (query row, query head).  Keys are walked from the first visible one in blocks of 32, a lane a key:
 // s_j = (q . k_j) * scale in 32-bit, a streaming softmax (running maximum m, sum l, accumulator acc; the sink is the
@@ -43,7 +44,7 @@ constexpr int kWarps = 4;
 enum MaskKind : int { MASK_CAUSAL = 0, MASK_WINDOW = 1, MASK_BLOCKS = 2, MASK_WINDOW_POOLED = 3 };
 
 // What only some mixers use: a learned sink score per query head (null: none, or the fixed 0 of `sink`), a cap on the
-// scores (0: none), the pooled blocks of MASK_WINDOW_POOLED (their pages, the requests' tables of those pages and
+// scores (0: none), a gate per row and head on the output, the pooled blocks of MASK_WINDOW_POOLED (their pages, the requests' tables of those pages and
 // the tokens a block holds), the first positions that MASK_WINDOW keeps, and the distance bias's two numbers per query
 // head (null: none).
 struct MaskExtras {
@@ -54,7 +55,15 @@ struct MaskExtras {
     int pool_bt_stride, pool;
     int keep_first;
     const float *bias_weight, *bias_rate;
+    const void* head_gate;            // [rows, heads] in the dtype of q (null: none), row stride head_gate_stride
+    int64_t head_gate_stride;
 };
+
+template <typename T>
+__device__ __forceinline__ float head_factor(const MaskExtras& x, int row, int head) {
+    if (x.head_gate == nullptr) return 1.0f;
+    return 1.0f / (1.0f + expf(-Elem<T>::load(reinterpret_cast<const T*>(x.head_gate) + (int64_t)row * x.head_gate_stride + head)));
+}
 
 __device__ __forceinline__ float capped(float s, float softcap) {
     return softcap > 0.0f ? softcap * tanhf(s / softcap) : s;
@@ -188,14 +197,14 @@ attention_masked_kernel(const T* __restrict__ q, int64_t q_stride, const T* __re
         }
         m = m_new;
     }
-    const float denom = fmaxf(l, 1.0e-30f);
+    const float denom = fmaxf(l, 1.0e-30f), whole = head_factor<T>(extras, row, head);
     const int64_t oat = (int64_t)row * out_stride + (int64_t)head * vdim;
     const T* grow = gate == nullptr ? nullptr : gate + (int64_t)row * gate_stride + (int64_t)head * vdim;
 #pragma unroll
     for (int c = 0; c < NCV; ++c) {
         const int col = c * 32 + lane;
         if (col < vdim) {
-            float value = acc[c] / denom;
+            float value = acc[c] / denom * whole;
             if (grow != nullptr) value *= 1.0f / (1.0f + expf(-Elem<T>::load(grow + col)));
             if (out_f32) reinterpret_cast<float*>(out)[oat + col] = value;
             else Elem<T>::store(out + oat + col, value);
@@ -403,7 +412,7 @@ attention_masked_packets_kernel(const T* __restrict__ q, int64_t q_stride, const
     if (vg != 0) return;
 #pragma unroll
     for (int h = 0; h < HPW; ++h) {
-        const float inv = 1.0f / fmaxf(l[h], 1.0e-30f);
+        const float inv = head_factor<T>(extras, row, head0 + h) / fmaxf(l[h], 1.0e-30f);
         const int64_t oat = (int64_t)row * out_stride + (int64_t)(head0 + h) * vdim;
         const T* grow = gate == nullptr ? nullptr : gate + (int64_t)row * gate_stride + (int64_t)(head0 + h) * vdim;
 #pragma unroll
@@ -536,14 +545,16 @@ int launch(const void* q, int64_t q_stride, const void* gate, int64_t gate_strid
 // 3 window with pooled blocks (pool_cache: the layer's pages of averaged keys and values, pool_table: the requests'
 // tables of those pages with row stride pool_bt_stride, pool: tokens a block).  sinks: null or float32 [heads];
 // softcap: 0 for none.  keep_first: first positions that a window (kind 1) keeps; bias_weight, bias_rate: null or float32
-// [heads] (not with pooled blocks).
+// [heads] (not with pooled blocks).  head_gate: null or [rows, heads] in `dtype`, row stride head_gate_stride: logits whose sigmoid
+// multiplies a head's output.
 TB_EXPORT int tb_attention_masked(const void* q, int64_t q_stride, const void* gate, int64_t gate_stride, void* out,
                                   int64_t out_stride, const void* cache, const int* positions, const int* seq_of_row,
                                   const int* block_table, int bt_stride, int rows, int heads, int kv_heads, int dim,
                                   int vdim, int page_size, int mask_kind, int mask_size, int sink, float scale,
                                   int keys_per_value, int out_f32, const float* sinks, float softcap,
                                   const void* pool_cache, const int* pool_table, int pool_bt_stride, int pool, int keep_first,
-                                  const float* bias_weight, const float* bias_rate, int dtype, cudaStream_t stream) {
+                                  const float* bias_weight, const float* bias_rate, const void* head_gate,
+                                  int64_t head_gate_stride, int dtype, cudaStream_t stream) {
     if (rows == 0) return 0;
     if (keep_first < 0 || (keep_first > 0 && mask_kind != MASK_WINDOW)) return TB_ERR_BAD_SIZE;
     if ((bias_weight == nullptr) != (bias_rate == nullptr) || (bias_weight != nullptr && mask_kind == MASK_WINDOW_POOLED))
@@ -555,6 +566,7 @@ TB_EXPORT int tb_attention_masked(const void* q, int64_t q_stride, const void* g
     extras.sinks = sinks; extras.softcap = softcap; extras.pool_cache = pool_cache; extras.pool_table = pool_table;
     extras.pool_bt_stride = pool_bt_stride; extras.pool = pool;
     extras.keep_first = keep_first; extras.bias_weight = bias_weight; extras.bias_rate = bias_rate;
+    extras.head_gate = head_gate; extras.head_gate_stride = head_gate_stride;
     if (dim < 1 || dim > 1024 || vdim < 1 || vdim > 512) return TB_ERR_BAD_SIZE;
     if (kv_heads < 1 || heads < 1 || heads % kv_heads != 0 || page_size < 1) return TB_ERR_BAD_SIZE;
     if (mask_kind < MASK_CAUSAL || mask_kind > MASK_WINDOW_POOLED) return TB_ERR_BAD_SIZE;

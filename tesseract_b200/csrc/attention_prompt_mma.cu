@@ -1,7 +1,8 @@
 // Paged attention on the tensor cores, for prompt portions and (second kernel) for steps of few rows, with 32-bit
 // scores and weights kept to 32-bit accuracy: the masks and page layout of attention_masked.cu (keys and values of separate widths; causal, sliding window or
 // blocks of positions, or a window with averaged blocks in front of it, which are walked first, from pages of their
-// own), its kept first positions, its learned sink per query head, its cap on the scores and its distance bias, for
+// own), its kept first positions, its learned sink per query head, its cap on the scores, its distance bias and its gate
+// per row and head, for
 // bfloat16 queries, keys and values.
 //
 //   S = Q K^T      mma.sync m16n8k16 on bfloat16 operands with 32-bit accumulators: the products of two bfloat16
@@ -38,7 +39,14 @@ struct Extras {
     int pool_bt_stride, pool;
     int keep_first;
     const float *bias_weight, *bias_rate;
+    const bf16* head_gate;                // [rows, heads] logits whose sigmoid multiplies a head's output (null: none)
+    int64_t head_gate_stride;
 };
+
+__device__ __forceinline__ float head_factor(const Extras& x, int row, int head) {
+    if (x.head_gate == nullptr) return 1.0f;
+    return 1.0f / (1.0f + __expf(-__bfloat162float(x.head_gate[(int64_t)row * x.head_gate_stride + head])));
+}
 
 // softcap * tanh(s / softcap) as softcap - 2 softcap / (2^(s k) + 1) with k = 2 log2(e) / softcap: one exponential and
 // one reciprocal of the fast kind, good to some 1e-6 of softcap, which is far below what the bfloat16 queries and keys
@@ -323,7 +331,7 @@ attention_prompt_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __re
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
         if (!there[r]) continue;
-        const float inv = 1.0f / fmaxf(l[r], 1.0e-30f);
+        const float inv = head_factor(x, r0 + i0 + g + r * 8, head) / fmaxf(l[r], 1.0e-30f);
         if (out_f32) {                                            // the weighted sums as they are, unrounded
             float* orow = reinterpret_cast<float*>(out) + (int64_t)(r0 + i0 + g + r * 8) * out_stride + (int64_t)head * DV;
 #pragma unroll
@@ -544,6 +552,7 @@ attention_rows_kernel(const bf16* __restrict__ q, int64_t q_stride, bf16* __rest
             value = fmaf(theirs[col], weight, value);
         }
         const int64_t at = (int64_t)row * out_stride + (int64_t)(kv_head * per + head_row) * DV + col;
+        value *= head_factor(x, row, kv_head * per + head_row);
         if (out_f32) reinterpret_cast<float*>(out)[at] = value / fmaxf(total, 1.0e-30f);
         else out[at] = __float2bfloat16_rn(value / fmaxf(total, 1.0e-30f));
     }
@@ -606,13 +615,15 @@ TB_EXPORT int tb_attention_prompt_mma_supported(int dim, int vdim) {
 // averages, pool_table: the requests' tables of those pages with row stride pool_bt_stride, pool: tokens a block).
 // sinks: null or float32 [heads]; softcap: 0 for none; keep_first: first positions that a window (kind 1) keeps; bias_weight,
 // bias_rate: null or float32 [heads] (a key at distance n loses bias_weight * ln(1 + bias_rate * n); not with pooled blocks).
+// head_gate: null or bfloat16 [rows, heads], row stride head_gate_stride.
 TB_EXPORT int tb_attention_prompt_mma(const void* q, int64_t q_stride, void* out, int64_t out_stride, const void* cache,
                                       const int* positions, const int* row_start, const int* block_table, int bt_stride,
                                       int rows, int num_seqs, int heads, int kv_heads, int dim, int vdim, int page_size,
                                       int mask_kind, int mask_size, float scale, int keys_per_value, int out_f32,
                                       const float* sinks, float softcap, const void* pool_cache, const int* pool_table,
                                       int pool_bt_stride, int pool, int keep_first, const float* bias_weight,
-                                      const float* bias_rate, cudaStream_t stream) {
+                                      const float* bias_rate, const void* head_gate, int64_t head_gate_stride,
+                                      cudaStream_t stream) {
     if (rows == 0) return 0;
     if (!extras_fit(mask_kind, keep_first, bias_weight, bias_rate)) return TB_ERR_BAD_SIZE;
     if (mask_kind == MASK_WINDOW_POOLED && (pool < 1 || pool_cache == nullptr || pool_table == nullptr || keys_per_value != 1 ||
@@ -623,6 +634,7 @@ TB_EXPORT int tb_attention_prompt_mma(const void* q, int64_t q_stride, void* out
     x.sinks = sinks; x.softcap = softcap; x.cap_k = softcap > 0.0f ? 2.8853900817779268f / softcap : 0.0f; x.pool_cache = (const bf16*)pool_cache; x.pool_table = pool_table;
     x.pool_bt_stride = pool_bt_stride; x.pool = pool;
     x.keep_first = keep_first; x.bias_weight = bias_weight; x.bias_rate = bias_rate;
+    x.head_gate = (const bf16*)head_gate; x.head_gate_stride = head_gate_stride;
     if (!tb_attention_prompt_mma_supported(dim, vdim)) return TB_ERR_BAD_SIZE;
     if (kv_heads < 1 || heads < 1 || heads % kv_heads != 0 || page_size < 1 || num_seqs < 1) return TB_ERR_BAD_SIZE;
     if (keys_per_value < 1 || kv_heads % keys_per_value != 0) return TB_ERR_BAD_SIZE;
@@ -650,7 +662,7 @@ TB_EXPORT int tb_attention_rows_mma(const void* q, int64_t q_stride, void* out, 
                                     int mask_size, float scale, int keys_per_value, int out_f32, const float* sinks,
                                     float softcap, const void* pool_cache, const int* pool_table, int pool_bt_stride,
                                     int pool, int keep_first, const float* bias_weight, const float* bias_rate,
-                                    cudaStream_t stream) {
+                                    const void* head_gate, int64_t head_gate_stride, cudaStream_t stream) {
     if (rows == 0) return 0;
     if (!extras_fit(mask_kind, keep_first, bias_weight, bias_rate)) return TB_ERR_BAD_SIZE;
     if (mask_kind == MASK_WINDOW_POOLED && (pool < 1 || pool_cache == nullptr || pool_table == nullptr || keys_per_value != 1 ||
@@ -661,6 +673,7 @@ TB_EXPORT int tb_attention_rows_mma(const void* q, int64_t q_stride, void* out, 
     x.sinks = sinks; x.softcap = softcap; x.cap_k = softcap > 0.0f ? 2.8853900817779268f / softcap : 0.0f; x.pool_cache = (const bf16*)pool_cache; x.pool_table = pool_table;
     x.pool_bt_stride = pool_bt_stride; x.pool = pool;
     x.keep_first = keep_first; x.bias_weight = bias_weight; x.bias_rate = bias_rate;
+    x.head_gate = (const bf16*)head_gate; x.head_gate_stride = head_gate_stride;
     if (!tb_attention_prompt_mma_supported(dim, vdim)) return TB_ERR_BAD_SIZE;
     if (kv_heads < 1 || heads < 1 || heads % kv_heads != 0 || heads / kv_heads > 16 || page_size < 1) return TB_ERR_BAD_SIZE;
     if (keys_per_value < 1 || kv_heads % keys_per_value != 0) return TB_ERR_BAD_SIZE;

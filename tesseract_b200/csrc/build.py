@@ -67,6 +67,8 @@ SOURCES: Dict[str, List[str]] = {
     "gated_residual": [],
     "short_conv": [],
     "rglru": [],
+    "hyper_streams": [],
+    "matrix_recurrence": [],
 }
 
 

@@ -17,6 +17,11 @@
 // 16-byte packet of the row.  All arithmetic is 32-bit; each stored value is rounded once; the order
 // of a head's sum of squares depends on d alone.
 //
+// tb_row_norm_rope_cache, for a mixer that norms its queries and its keys over the whole projection (all heads at once, a weight
+// per number) in front of the rotation, does the same job with a block a row: the sums of squares of the row's q and of its k, the
+// normed numbers turned with the row's sines and cosines (taken once a row), stored; the values are the row's own value columns
+// or, with `values_from_keys`, the keys as projected (dv = d, no value columns).
+//
 // tb_pool_blocks, for a mixer that also attends to averaged blocks of old tokens, runs behind it: every row that ends a
 // block of `pool` positions leaves the block's averaged key and value in pages of their own.
 #include "common.cuh"
@@ -214,6 +219,101 @@ int launch_rope_norm(const void* proj, int64_t proj_stride, void* q_out, int64_t
     return launched == cudaSuccess ? tb_launch_status() : (int)launched;
 }
 
+// q and k of a row over their own root mean squares (all heads at once) times a weight, then the rotation; a block a row, the
+// row's q and k widened in shared memory.  VEC: stores of a 16-byte packet (head sizes and half rotations that are multiples of a
+// packet, or no rotation).
+constexpr int kRowThreads = 256;
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kRowThreads)
+row_norm_rope_cache_kernel(const T* __restrict__ proj, int64_t proj_stride, T* __restrict__ q_out, int64_t q_stride,
+                           T* __restrict__ cache, const int* __restrict__ positions, const int* __restrict__ seq_of_row,
+                           const int* __restrict__ block_table, int bt_stride, const float* __restrict__ inv_freq,
+                           const float* __restrict__ weight, HeadGeometry g, int values_from_keys) {
+    extern __shared__ __align__(16) float row_smem[];  // [q_width + k_width] numbers, then [half] cosines, [half] sines
+    __shared__ float scratch[32];
+    constexpr int N = VEC ? Packet<T>::N : 1;
+    pdl_trigger();
+    pdl_wait();
+    const int row = blockIdx.x, pos = positions[row];
+    const int q_width = g.heads * g.dim, both = q_width + g.kv_heads * g.dim, half = g.rot_dims >> 1;
+    float *cosines = row_smem + both, *sines = cosines + half;
+    const T* prow = proj + (int64_t)row * proj_stride;
+    float qq = 0.0f, kk = 0.0f;
+    for (int i = threadIdx.x * N; i < both; i += kRowThreads * N) {
+        float v[N];
+        if constexpr (VEC) Packet<T>::load(prow + i, v);
+        else v[0] = Elem<T>::load(prow + i);
+        float sum = 0.0f;
+#pragma unroll
+        for (int e = 0; e < N; ++e) {
+            row_smem[i + e] = v[e];
+            sum = fmaf(v[e], v[e], sum);
+        }
+        if (i < q_width) qq += sum; else kk += sum;    // (a packet does not straddle: widths are multiples of a head)
+    }
+    for (int i = threadIdx.x; i < half; i += kRowThreads) {
+        float sn, cs;
+        sincosf((float)pos * inv_freq[i], &sn, &cs);
+        cosines[i] = cs * g.amplitude;
+        sines[i] = sn * g.amplitude;
+    }
+    const float inv_q = 1.0f / sqrtf(block_sum(qq, scratch) / (float)q_width + g.eps);
+    const float inv_k = 1.0f / sqrtf(block_sum(kk, scratch) / (float)(both - q_width) + g.eps);
+    __syncthreads();
+    const int page = block_table[(int64_t)seq_of_row[row] * bt_stride + pos / g.page_size], in_page = pos % g.page_size;
+    T* keys = cache + (int64_t)page * g.kv_heads * g.page_size * (g.dim + g.vdim);
+    T* values = keys + (int64_t)g.kv_heads * g.page_size * g.dim;
+    for (int i = threadIdx.x * N; i < both; i += kRowThreads * N) {
+        const bool is_key = i >= q_width;
+        const int head = (is_key ? i - q_width : i) / g.dim, at = (is_key ? i - q_width : i) % g.dim;
+        const float inv = is_key ? inv_k : inv_q;
+        float v[N];
+#pragma unroll
+        for (int e = 0; e < N; ++e) v[e] = row_smem[i + e] * inv * weight[i + e];
+        if (at < g.rot_dims) {                         // (with VEC a packet lies wholly in one half)
+            const bool second = at >= half;
+            const int other = second ? i - half : i + half, angle = second ? at - half : at;
+#pragma unroll
+            for (int e = 0; e < N; ++e) {
+                const float w = row_smem[other + e] * inv * weight[other + e];
+                v[e] = second ? v[e] * cosines[angle + e] + w * sines[angle + e] : v[e] * cosines[angle + e] - w * sines[angle + e];
+            }
+        }
+        T* dst = is_key ? keys + ((int64_t)head * g.page_size + in_page) * g.dim + at : q_out + (int64_t)row * q_stride + i;
+        if constexpr (VEC) Packet<T>::store(dst, v);
+        else Elem<T>::store(dst, v[0]);
+    }
+    const int v_width = g.kv_heads * g.vdim;
+    const T* src = values_from_keys ? prow + q_width : prow + both;
+    for (int i = threadIdx.x * N; i < v_width; i += kRowThreads * N) {
+        T* dst = values + ((int64_t)(i / g.vdim) * g.page_size + in_page) * g.vdim + i % g.vdim;
+        if constexpr (VEC) *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src + i);
+        else *dst = src[i];
+    }
+}
+
+template <typename T>
+int launch_row_norm(const void* proj, int64_t proj_stride, void* q_out, int64_t q_stride, void* cache, const int* positions,
+                    const int* seq_of_row, const int* block_table, int bt_stride, const float* inv_freq, const float* weight,
+                    int rows, const HeadGeometry& g, int values_from_keys, cudaStream_t stream) {
+    constexpr int N = Packet<T>::N;
+    const uintptr_t bits = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache;
+    const bool vec = g.dim % N == 0 && g.vdim % N == 0 && (g.rot_dims / 2) % N == 0 && proj_stride % N == 0 && q_stride % N == 0 &&
+                     bits % 16 == 0;
+    const size_t smem = sizeof(float) * ((size_t)(g.heads + g.kv_heads) * g.dim + g.rot_dims);
+    if (smem > 200 * 1024) return TB_ERR_BAD_SIZE;
+    auto kernel = vec ? row_norm_rope_cache_kernel<T, true> : row_norm_rope_cache_kernel<T, false>;
+    if (smem > 40 * 1024) {
+        cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (err != cudaSuccess) return (int)err;
+    }
+    cudaError_t launched = tb_launch_pdl(kernel, dim3(rows), dim3(kRowThreads), smem, stream, (const T*)proj, proj_stride,
+                                         (T*)q_out, q_stride, (T*)cache, positions, seq_of_row, block_table, bt_stride, inv_freq,
+                                         weight, g, values_from_keys);
+    return launched == cudaSuccess ? tb_launch_status() : (int)launched;
+}
+
 // For every row of the step that ends a block of `pool` positions ((position + 1) % pool == 0): the averages of the block's
 // keys and of its values, as the pages hold them, into entry position / pool of the request's pooled pages (same page
 // layout).  A block of threads per (row, kv head), a thread a column, the block's tokens added in order in 32-bit.
@@ -285,6 +385,29 @@ TB_EXPORT int tb_rope_norm_cache(const void* proj, int64_t proj_stride, void* q_
     if (dtype == TB_BF16)
         return launch_rope_norm<__nv_bfloat16>(proj, proj_stride, q_out, q_stride, cache, positions, seq_of_row, block_table,
                                                bt_stride, inv_freq, bias, rows, g, write_kv, values, stream);
+    return TB_ERR_BAD_DTYPE;
+}
+
+// proj: [rows, >= (H + G) * d (+ G * dv)] with row stride proj_stride; weight: 32-bit [(H + G) * d], the norm's weights of q then of k;
+// values_from_keys: dv = d and the values are the keys as projected.  The rest as for tb_rope_norm_cache.
+TB_EXPORT int tb_row_norm_rope_cache(const void* proj, int64_t proj_stride, void* q_out, int64_t q_stride, void* cache,
+                                     const int* positions, const int* seq_of_row, const int* block_table, int bt_stride,
+                                     const float* inv_freq, const float* weight, float amplitude, int rows, int heads, int kv_heads,
+                                     int dim, int vdim, int rot_dims, float eps, int page_size, int values_from_keys, int dtype,
+                                     cudaStream_t stream) {
+    if (rows == 0) return 0;
+    if (heads < 1 || kv_heads < 1 || dim < 1 || vdim < 1 || page_size < 1 || weight == nullptr) return TB_ERR_BAD_SIZE;
+    if (rot_dims < 0 || rot_dims > dim || rot_dims % 2 != 0 || (rot_dims > 0 && inv_freq == nullptr)) return TB_ERR_BAD_SIZE;
+    if (values_from_keys && dim != vdim) return TB_ERR_BAD_SIZE;
+    HeadGeometry g;
+    g.heads = heads; g.kv_heads = kv_heads; g.dim = dim; g.vdim = vdim; g.rot_dims = rot_dims; g.page_size = page_size;
+    g.unit_norm = 0; g.amplitude = amplitude; g.eps = eps;
+    if (dtype == TB_F32)
+        return launch_row_norm<float>(proj, proj_stride, q_out, q_stride, cache, positions, seq_of_row, block_table, bt_stride,
+                                      inv_freq, weight, rows, g, values_from_keys, stream);
+    if (dtype == TB_BF16)
+        return launch_row_norm<__nv_bfloat16>(proj, proj_stride, q_out, q_stride, cache, positions, seq_of_row, block_table,
+                                              bt_stride, inv_freq, weight, rows, g, values_from_keys, stream);
     return TB_ERR_BAD_DTYPE;
 }
 

@@ -3,6 +3,7 @@
 //
 //   tb_short_conv        v[t, c] = proj[t, c] + in_bias[c]                       (in_bias may be null)
 //                        y[t, c] = out_bias[c] + sum_{j < J} taps[j, c] * v[t - (J - 1) + j, c]     (out_bias may be null)
+//                        and y <- silu(y) with `act`;
 //                        with v = 0 at positions in front of the sequence's start.  Values at positions in front of this
 //                        step's first token come from the request's convolution state: the last J - 1 rows of v, 32-bit,
 //                        [slot][J - 1][channels]; position p lies at index p - (begin - (J - 1)).
@@ -17,6 +18,8 @@
 
 namespace {
 
+__device__ __forceinline__ float activated(float y, int act) { return act ? y / (1.0f + expf(-y)) : y; }
+
 // A thread a (row, channel): any width, any number of taps.
 template <typename T, bool SINGLE>
 __global__ void __launch_bounds__(128)
@@ -24,7 +27,7 @@ short_conv_kernel(const T* __restrict__ proj, int64_t proj_stride, const float* 
                   const float* __restrict__ taps, const float* __restrict__ out_bias, float* __restrict__ state,
                   T* __restrict__ out, int64_t out_stride, const int* __restrict__ positions,
                   const int* __restrict__ seq_of_row, const int* __restrict__ row_start, const int* __restrict__ seq_begin,
-                  const int* __restrict__ state_slots, int channels, int J) {
+                  const int* __restrict__ state_slots, int channels, int J, int act) {
     pdl_trigger();
     pdl_wait();                                   // the projected rows and the step's metadata come from kernels in front
     const int row = blockIdx.x;
@@ -44,7 +47,7 @@ short_conv_kernel(const T* __restrict__ proj, int64_t proj_stride, const float* 
         if (SINGLE && j > 0) st[(int64_t)(j - 1) * channels] = v;      // (index j - 1 has been read: the walk ascends)
     }
     if (out_bias != nullptr) sum += out_bias[c];
-    Elem<T>::store(out + (int64_t)row * out_stride + c, sum);
+    Elem<T>::store(out + (int64_t)row * out_stride + c, activated(sum, act));
 }
 
 template <int N>
@@ -71,7 +74,8 @@ short_conv_packets_kernel(const T* __restrict__ proj, int64_t proj_stride, const
                           const float* __restrict__ taps, const float* __restrict__ out_bias, float* __restrict__ state,
                           T* __restrict__ out, int64_t out_stride, const int* __restrict__ positions,
                           const int* __restrict__ seq_of_row, const int* __restrict__ row_start,
-                          const int* __restrict__ seq_begin, const int* __restrict__ state_slots, int channels, int rows) {
+                          const int* __restrict__ seq_begin, const int* __restrict__ state_slots, int channels, int rows,
+                          int act) {
     constexpr int N = Packet<T>::N;
     constexpr int ROWS = SINGLE ? 1 : kRowTile;
     const int packet = blockIdx.y * blockDim.x + threadIdx.x;
@@ -137,7 +141,7 @@ short_conv_packets_kernel(const T* __restrict__ proj, int64_t proj_stride, const
             float sum = 0.0f;
 #pragma unroll
             for (int j = 0; j < J; ++j) sum = fmaf(w[j][e], v[j][e], sum);
-            y[e] = sum + behind[e];
+            y[e] = activated(sum + behind[e], act);
         }
         if (SINGLE) {
 #pragma unroll
@@ -175,7 +179,7 @@ short_conv_state_kernel(const T* __restrict__ proj, int64_t proj_stride, const f
 template <typename T>
 int launch(const void* proj, int64_t proj_stride, const float* in_bias, const float* taps, const float* out_bias,
            float* state, void* out, int64_t out_stride, const int* positions, const int* seq_of_row, const int* row_start,
-           const int* seq_begin, const int* state_slots, int rows, int channels, int J, int single, cudaStream_t stream) {
+           const int* seq_begin, const int* state_slots, int rows, int channels, int J, int single, int act, cudaStream_t stream) {
     constexpr int N = Packet<T>::N;
     const uintptr_t bits = (uintptr_t)proj | (uintptr_t)in_bias | (uintptr_t)taps | (uintptr_t)out_bias | (uintptr_t)state |
                            (uintptr_t)out;
@@ -186,7 +190,7 @@ int launch(const void* proj, int64_t proj_stride, const float* in_bias, const fl
 #define TB_CONV(S, TAPS)                                                                                              \
     launched = tb_launch_pdl(short_conv_packets_kernel<T, S, TAPS>, grid, dim3(128), 0, stream, (const T*)proj,       \
                              proj_stride, in_bias, taps, out_bias, state, (T*)out, out_stride, positions, seq_of_row, \
-                             row_start, seq_begin, state_slots, channels, rows)
+                             row_start, seq_begin, state_slots, channels, rows, act)
         if (single) {
             if (J == 1) TB_CONV(true, 1); else if (J == 2) TB_CONV(true, 2); else if (J == 3) TB_CONV(true, 3); else TB_CONV(true, 4);
         } else {
@@ -198,7 +202,7 @@ int launch(const void* proj, int64_t proj_stride, const float* in_bias, const fl
         auto kernel = single ? short_conv_kernel<T, true> : short_conv_kernel<T, false>;
         launched = tb_launch_pdl(kernel, grid, dim3(128), 0, stream, (const T*)proj, proj_stride, in_bias, taps, out_bias,
                                  state, (T*)out, out_stride, positions, seq_of_row, row_start, seq_begin, state_slots,
-                                 channels, J);
+                                 channels, J, act);
     }
     return launched == cudaSuccess ? tb_launch_status() : (int)launched;
 }
@@ -207,21 +211,21 @@ int launch(const void* proj, int64_t proj_stride, const float* in_bias, const fl
 
 // proj: [rows, channels] with row stride proj_stride (elements); taps: 32-bit [J, channels] (tap J - 1 multiplies the row
 // itself, tap 0 the oldest); in_bias, out_bias: null or 32-bit [channels]; state: 32-bit [slots, J - 1, channels] (null
-// for one tap); out: [rows, channels] in the dtype of proj.
+// for one tap); out: [rows, channels] in the dtype of proj; act: 1 applies SiLU to the sums.
 TB_EXPORT int tb_short_conv(const void* proj, int64_t proj_stride, const float* in_bias, const float* taps,
                             const float* out_bias, float* state, void* out, int64_t out_stride, const int* positions,
                             const int* seq_of_row, const int* row_start, const int* seq_begin, const int* state_slots,
-                            int rows, int channels, int taps_count, int single, int dtype, cudaStream_t stream) {
+                            int rows, int channels, int taps_count, int single, int act, int dtype, cudaStream_t stream) {
     if (rows == 0) return 0;
     if (channels < 1 || taps_count < 1 || (channels + 127) / 128 > 65535) return TB_ERR_BAD_SIZE;
     if (taps_count > 1 && state == nullptr) return TB_ERR_BAD_SIZE;
     if (dtype == TB_F32)
         return launch<float>(proj, proj_stride, in_bias, taps, out_bias, state, out, out_stride, positions, seq_of_row,
-                             row_start, seq_begin, state_slots, rows, channels, taps_count, single, stream);
+                             row_start, seq_begin, state_slots, rows, channels, taps_count, single, act, stream);
     if (dtype == TB_BF16)
         return launch<__nv_bfloat16>(proj, proj_stride, in_bias, taps, out_bias, state, out, out_stride, positions,
                                      seq_of_row, row_start, seq_begin, state_slots, rows, channels, taps_count, single,
-                                     stream);
+                                     act, stream);
     return TB_ERR_BAD_DTYPE;
 }
 

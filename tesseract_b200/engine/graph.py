@@ -45,6 +45,8 @@ def graph_safe(model) -> bool:
             parts.append(block.token_input)
         if getattr(block, "gates", None) is not None:
             parts.append(block.gates)
+        if getattr(block, "mixing", None) is not None:
+            parts.append(block.mixing)
     return all(getattr(part, "graph_safe", False) for part in parts)
 
 

@@ -74,7 +74,7 @@ def make_stepper(model: DecoderModel, *, capacity_tokens: int, page_size: int = 
                  max_step_tokens: int = 4096) -> Stepper:
     """A cache sized for ``capacity_tokens`` and the step function over it."""
     needs = model.cache_needs()
-    cache_of = [entry.cache_of for entry in model.spec.run_order]
+    cache_of = model.cache_sources()
     num_pages = max(1, -(-capacity_tokens // page_size))
     cache = CacheManager(needs, cache_of, num_pages=num_pages, page_size=page_size, max_requests=max_requests,
                          dtype=model.runtime.dtype, device=model.runtime.device, max_step_tokens=max_step_tokens)

@@ -813,7 +813,8 @@ def attention_masked(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
                      positions: torch.Tensor, seq_of_row: torch.Tensor, block_table: torch.Tensor, *, heads: int,
                      kv_heads: int, dim: int, vdim: int, page_size: int, mask_kind: int, mask_size: int, sink: bool,
                      scale: float, keys_per_value: int = 1, sinks: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                     pooled=None, keep_first: int = 0, distance_bias=None) -> torch.Tensor:
+                     pooled=None, keep_first: int = 0, distance_bias=None,
+                     head_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Paged attention with 32-bit scores and weights: ``q`` ``[T, heads * dim]``, optional ``gate``
     ``[T, heads * vdim]`` (the output is multiplied by its sigmoid), ``out`` ``[T, heads * vdim]`` in the dtype of ``q``
     or in float32 (the weighted sums as they are, unrounded); pages hold ``[kv_heads, page_size, dim]`` keys then
@@ -825,7 +826,8 @@ def attention_masked(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
     denominator, or, with ``sinks`` (float32 ``[heads]``), of a learned score per head; ``softcap`` > 0: a score ``s``
     becomes ``softcap * tanh(s / softcap)``; ``keep_first`` (with ``MASK_WINDOW``): the first positions of the sequence that
     every row sees although its window has passed them; ``distance_bias = (weight, rate)`` (float32 ``[heads]`` each): the
-    score of the key ``n`` positions back loses ``weight * ln(1 + rate * n)``."""
+    score of the key ``n`` positions back loses ``weight * ln(1 + rate * n)``; ``head_gate`` (``[T, heads]``, the dtype of ``q``):
+    head ``h``'s output is multiplied by the sigmoid of its number."""
     _cuda(q, gate, out, cache, positions, seq_of_row, block_table)
     rows = q.shape[0]
     _need(q.stride(1) == 1 and q.shape[1] == heads * dim, "attention_masked q")
@@ -836,7 +838,7 @@ def attention_masked(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
     _need(cache.dtype == q.dtype and cache.is_contiguous(), "attention_masked cache")
     if gate is not None:
         _need(gate.stride(1) == 1 and gate.shape == (rows, heads * vdim) and gate.dtype == q.dtype, "attention_masked gate")
-    extras = _mask_extras("attention_masked", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias)
+    extras = _mask_extras("attention_masked", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias, head_gate)
     lib = load_library("attention_masked")
     _check(lib.tb_attention_masked(_ptr(q), _i64(q.stride(0)), _ptr(gate), _i64(gate.stride(0) if gate is not None else 0),
                                    _ptr(out), _i64(out.stride(0)), _ptr(cache), _ptr(positions), _ptr(seq_of_row),
@@ -849,9 +851,9 @@ def attention_masked(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.T
 
 
 def _mask_extras(what: str, q: torch.Tensor, heads: int, mask_kind: int, keys_per_value: int, sinks, pooled, keep_first,
-                 distance_bias):
-    """The arguments that a learned sink, pooled blocks, kept first positions and a distance bias add to an attention
-    kernel's call, checked."""
+                 distance_bias, head_gate):
+    """The arguments that a learned sink, pooled blocks, kept first positions, a distance bias and a gate per head add to an
+    attention kernel's call, checked."""
     weight = rate = None
     if distance_bias is not None:
         weight, rate = distance_bias
@@ -859,6 +861,10 @@ def _mask_extras(what: str, q: torch.Tensor, heads: int, mask_kind: int, keys_pe
         for v in (weight, rate):
             _need(v.dtype == torch.float32 and v.numel() == heads and v.is_contiguous(), f"{what} distance bias")
     _need(keep_first == 0 or (keep_first > 0 and mask_kind == MASK_WINDOW), f"{what}: only a window keeps first positions")
+    if head_gate is not None:
+        _cuda(head_gate)
+        _need(head_gate.dtype == q.dtype and head_gate.stride(1) == 1 and tuple(head_gate.shape) == (q.shape[0], heads),
+              f"{what} head gate")
     if sinks is not None:
         _cuda(sinks)
         _need(sinks.dtype == torch.float32 and sinks.numel() == heads and sinks.is_contiguous(), f"{what} sinks")
@@ -871,7 +877,8 @@ def _mask_extras(what: str, q: torch.Tensor, heads: int, mask_kind: int, keys_pe
         _need(pool_cache.dtype == q.dtype and pool_cache.is_contiguous() and pool_table.dtype == torch.int32
               and pool_table.stride(1) == 1 and pool >= 1, f"{what} pooled pages")
     return (_ptr(pool_cache), _ptr(pool_table), _i32(pool_table.stride(0) if pool_table is not None else 0), _i32(pool),
-            _i32(keep_first), _ptr(weight), _ptr(rate))
+            _i32(keep_first), _ptr(weight), _ptr(rate), _ptr(head_gate),
+            _i64(head_gate.stride(0) if head_gate is not None else 0))
 
 
 def attention_prompt_mma_supported(dtype: torch.dtype, dim: int, vdim: int) -> bool:
@@ -884,7 +891,8 @@ def attention_prompt_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor
                          row_start: torch.Tensor, block_table: torch.Tensor, *, num_seqs: int, heads: int,
                          kv_heads: int, dim: int, vdim: int, page_size: int, mask_kind: int, mask_size: int,
                          scale: float, keys_per_value: int = 1, sinks: Optional[torch.Tensor] = None,
-                         softcap: float = 0.0, pooled=None, keep_first: int = 0, distance_bias=None) -> torch.Tensor:
+                         softcap: float = 0.0, pooled=None, keep_first: int = 0, distance_bias=None,
+                         head_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """:func:`attention_masked` (no fixed sink, no gate; ``sinks``, ``softcap`` and ``pooled`` as there) for bfloat16 prompt portions on the tensor cores: scores from
     exact bfloat16 products with 32-bit accumulation, 32-bit softmax, the 32-bit weights split in two bfloat16 halves
     for the product with the values.  The rows of a sequence (``row_start``) stand at consecutive positions.  ``out`` in
@@ -897,7 +905,7 @@ def attention_prompt_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor
     _need(keys_per_value >= 1 and kv_heads % keys_per_value == 0, "attention_prompt_mma keys_per_value")
     _need(cache.dtype == q.dtype and cache.is_contiguous(), "attention_prompt_mma cache")
     _need(row_start.dtype == torch.int32 and row_start.numel() >= num_seqs + 1, "attention_prompt_mma row_start")
-    extras = _mask_extras("attention_prompt_mma", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias)
+    extras = _mask_extras("attention_prompt_mma", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias, head_gate)
     lib = load_library("attention_prompt_mma")
     _check(lib.tb_attention_prompt_mma(_ptr(q), _i64(q.stride(0)), _ptr(out), _i64(out.stride(0)), _ptr(cache),
                                        _ptr(positions), _ptr(row_start), _ptr(block_table), _i32(block_table.stride(0)),
@@ -913,7 +921,8 @@ def attention_rows_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
                        seq_of_row: torch.Tensor, block_table: torch.Tensor, *, heads: int, kv_heads: int, dim: int,
                        vdim: int, page_size: int, mask_kind: int, mask_size: int, scale: float,
                        keys_per_value: int = 1, sinks: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                       pooled=None, keep_first: int = 0, distance_bias=None) -> torch.Tensor:
+                       pooled=None, keep_first: int = 0, distance_bias=None,
+                       head_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """:func:`attention_prompt_mma` for steps of few rows at any positions: a block a (row, kv head), the kv head's
     query heads (at most 16) side by side in the tensor-core tile."""
     _cuda(q, out, cache, positions, seq_of_row, block_table)
@@ -923,7 +932,7 @@ def attention_rows_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
           "attention_rows_mma out")
     _need(keys_per_value >= 1 and kv_heads % keys_per_value == 0, "attention_rows_mma keys_per_value")
     _need(cache.dtype == q.dtype and cache.is_contiguous(), "attention_rows_mma cache")
-    extras = _mask_extras("attention_rows_mma", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias)
+    extras = _mask_extras("attention_rows_mma", q, heads, mask_kind, keys_per_value, sinks, pooled, keep_first, distance_bias, head_gate)
     lib = load_library("attention_prompt_mma")
     _check(lib.tb_attention_rows_mma(_ptr(q), _i64(q.stride(0)), _ptr(out), _i64(out.stride(0)), _ptr(cache),
                                      _ptr(positions), _ptr(seq_of_row), _ptr(block_table), _i32(block_table.stride(0)),
@@ -957,9 +966,9 @@ def gated_recurrence(proj: torch.Tensor, bias_z: torch.Tensor, bias_x: torch.Ten
 def short_conv(proj: torch.Tensor, in_bias: Optional[torch.Tensor], taps: torch.Tensor, out_bias: Optional[torch.Tensor],
                state: Optional[torch.Tensor], out: torch.Tensor, positions: torch.Tensor, seq_of_row: torch.Tensor,
                row_start: torch.Tensor, seq_begin: torch.Tensor, state_slots: torch.Tensor, *, num_seqs: int,
-               single: bool) -> torch.Tensor:
+               single: bool, activation: bool = False) -> torch.Tensor:
     """A causal convolution per channel of ``proj + in_bias`` (``[T, C]``; ``taps`` float32 ``[J, C]``, oldest first) plus
-    ``out_bias``; ``state`` (float32 ``[slots, J - 1, C]``; None for one tap) holds each request's last ``J - 1`` rows of
+    ``out_bias``, with ``activation`` through SiLU; ``state`` (float32 ``[slots, J - 1, C]``; None for one tap) holds each request's last ``J - 1`` rows of
     ``proj + in_bias`` and is renewed.  ``single``: every sequence brings one row (the state is renewed inside the kernel);
     otherwise a second launch renews it."""
     _cuda(proj, in_bias, taps, out_bias, state, out, positions, seq_of_row, row_start, seq_begin, state_slots)
@@ -979,7 +988,7 @@ def short_conv(proj: torch.Tensor, in_bias: Optional[torch.Tensor], taps: torch.
     _check(lib.tb_short_conv(_ptr(proj), _i64(proj.stride(0)), _ptr(in_bias), _ptr(taps), _ptr(out_bias), _ptr(state), _ptr(out),
                              _i64(out.stride(0)), _ptr(positions), _ptr(seq_of_row), _ptr(row_start), _ptr(seq_begin),
                              _ptr(state_slots), _i32(rows), _i32(channels), _i32(count), _i32(1 if single else 0),
-                             _i32(_code(proj.dtype)), _stream()), "short_conv")
+                             _i32(1 if activation else 0), _i32(_code(proj.dtype)), _stream()), "short_conv")
     if not single and count > 1:
         _check(lib.tb_short_conv_state(_ptr(proj), _i64(proj.stride(0)), _ptr(in_bias), _ptr(state), _ptr(row_start),
                                        _ptr(seq_begin), _ptr(state_slots), _i32(num_seqs), _i32(channels), _i32(count),
@@ -1272,6 +1281,36 @@ def rope_norm_cache(proj: torch.Tensor, q_out: torch.Tensor, cache: torch.Tensor
                                   _i32(vdim), _i32(rot_dims), _i32(1 if unit_norm else 0), _f32(eps), _i32(page_size),
                                   _i32(1 if write_kv else 0), _i32(value_mode), _ptr(first), _ptr(mix),
                                   _i32(_code(proj.dtype)), _stream()), "rope_norm_cache")
+
+
+def row_norm_rope_cache(proj: torch.Tensor, q_out: torch.Tensor, cache: torch.Tensor, positions: torch.Tensor,
+                        seq_of_row: torch.Tensor, block_table: torch.Tensor, inv_freq: Optional[torch.Tensor],
+                        weight: torch.Tensor, *, amplitude: float, heads: int, kv_heads: int, dim: int, vdim: int,
+                        rot_dims: int, eps: float, page_size: int, values_from_keys: bool) -> None:
+    """Queries and keys of ``proj`` (``[heads * dim | kv_heads * dim]``, then ``kv_heads * vdim`` values unless
+    ``values_from_keys``: the keys as projected are the values) over the root mean square of the whole row's q and of its k,
+    times ``weight`` (float32, q's numbers then k's), then the rotate-half rotation of :func:`rope_norm_cache`; stored as there."""
+    _cuda(proj, q_out, cache, positions, seq_of_row, block_table, inv_freq, weight)
+    rows = q_out.shape[0]
+    both = (heads + kv_heads) * dim
+    channels = both + (0 if values_from_keys else kv_heads * vdim)
+    _need(not values_from_keys or dim == vdim, "row_norm_rope_cache: keys that are values have their width")
+    _need(proj.stride(1) == 1 and proj.shape[1] >= channels and proj.shape[0] == rows, "row_norm_rope_cache proj")
+    _need(q_out.stride(1) == 1 and q_out.shape[1] == heads * dim and q_out.dtype == proj.dtype, "row_norm_rope_cache q_out")
+    _need(cache.dtype == proj.dtype and cache.is_contiguous(), "row_norm_rope_cache cache dtype")
+    _need(weight.dtype == torch.float32 and weight.numel() == both and weight.is_contiguous(), "row_norm_rope_cache weight")
+    if rot_dims:
+        _need(inv_freq is not None and inv_freq.dtype == torch.float32 and inv_freq.numel() == rot_dims // 2
+              and inv_freq.is_contiguous(), "row_norm_rope_cache inv_freq")
+    for t in (positions, seq_of_row, block_table):
+        _need(t.dtype == torch.int32, "row_norm_rope_cache metadata must be int32")
+    lib = load_library("rope_norm_cache")
+    _check(lib.tb_row_norm_rope_cache(_ptr(proj), _i64(proj.stride(0)), _ptr(q_out), _i64(q_out.stride(0)), _ptr(cache),
+                                      _ptr(positions), _ptr(seq_of_row), _ptr(block_table), _i32(block_table.stride(0)),
+                                      _ptr(inv_freq), _ptr(weight), _f32(amplitude), _i32(rows), _i32(heads), _i32(kv_heads),
+                                      _i32(dim), _i32(vdim), _i32(rot_dims), _f32(eps), _i32(page_size),
+                                      _i32(1 if values_from_keys else 0), _i32(_code(proj.dtype)), _stream()),
+           "row_norm_rope_cache")
 
 
 def pool_blocks(cache: torch.Tensor, pool_cache: torch.Tensor, positions: torch.Tensor, seq_of_row: torch.Tensor,
@@ -1692,4 +1731,138 @@ def attention_latent_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor
     if splits > 1:
         global launch_count
         launch_count += 1          # (the kernel that adds the runs up)
+    return out
+
+
+# ----------------------------------------------------------------------------- a stream of several copies
+
+
+def mixed_streams_norm(residual: torch.Tensor, update, mix: Optional[torch.Tensor], share: Optional[torch.Tensor],
+                       take: Optional[torch.Tensor], weight: Optional[torch.Tensor], out: Optional[torch.Tensor],
+                       streams: int, eps: float) -> None:
+    """``residual`` (float32 ``[T, S * W]``): ``S`` copies of a stream side by side.  With ``update = (a, scale_a, b, scale_b)``
+    (float32 ``[T, W]``, ``b`` may be None) every copy becomes ``x_t = sum_s mix[s, t] x_s + share[t] (scale_a a + scale_b b)``, in
+    place, all from the old ones; with ``out``, ``u = sum_s take[s] x_s`` and ``out = u / sqrt(mean(u^2) + eps) * weight``."""
+    rows = residual.shape[0]
+    width = residual.shape[1] // max(1, streams)
+    _cuda(residual, mix, share, take, weight, out)
+    _f32_rows(residual, (rows, streams * width), "mixed_streams_norm: the stream is contiguous float32 [rows, copies * width]")
+    a, scale_a, b, scale_b = update if update is not None else (None, 0.0, None, 0.0)
+    _cuda(a, b)
+    _f32_rows(a, (rows, width), "mixed_streams_norm update")
+    _f32_rows(b, (rows, width), "mixed_streams_norm update")
+    if a is not None:
+        _need(mix is not None and share is not None, "mixed_streams_norm: an update needs its weights")
+        _f32_rows(mix, (streams, streams), "mixed_streams_norm mix is float32 [copies, copies]")
+        _f32_rows(share, (streams,), "mixed_streams_norm share is float32 [copies]")
+    if out is not None:
+        _need(tuple(out.shape) == (rows, width) and out.is_contiguous() and take is not None and weight is not None,
+              "mixed_streams_norm out")
+        _f32_rows(take, (streams,), "mixed_streams_norm take is float32 [copies]")
+        _f32_rows(weight, (width,), "mixed_streams_norm weight is float32 [width]")
+    lib = load_library("hyper_streams")
+    _check(lib.tb_mixed_streams_norm(_ptr(residual), _ptr(a), _f32(scale_a), _ptr(b), _f32(scale_b), _ptr(mix), _ptr(share),
+                                     _ptr(take), _ptr(weight), _ptr(out), _i32(rows), _i32(width), _i32(streams), _f32(eps),
+                                     _i32(_code(out.dtype) if out is not None else 0), _stream()), "mixed_streams_norm")
+
+
+def bigram_embedding(tokens: torch.Tensor, positions: torch.Tensor, seq_of_row: torch.Tensor, row_start: torch.Tensor,
+                     state_slots: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, before: torch.Tensor,
+                     out: torch.Tensor, copies: int, mul_prev: int, mul_cur: int) -> torch.Tensor:
+    """``out[t]`` (float32 ``[T, copies * W]``) = ``copies`` times ``table[token] + pairs[h]`` with ``h = (token in front * mul_prev +
+    token * mul_cur) mod buckets`` and ``h = buckets`` (the last row of ``pairs`` ``[buckets + 1, W]``) at position 0.  ``before``
+    (int32 ``[slots]``) holds every request's last token and is renewed."""
+    _cuda(tokens, positions, seq_of_row, row_start, state_slots, table, pairs, before, out)
+    rows, width = out.shape[0], table.shape[1]
+    _f32_rows(out, (rows, copies * width), "bigram_embedding out is contiguous float32")
+    for t in (tokens, positions, seq_of_row, row_start, state_slots, before):
+        _need(t.dtype == torch.int32 and t.is_contiguous(), "bigram_embedding tokens, metadata and state are int32")
+    _need(tokens.numel() >= rows and positions.numel() >= rows and seq_of_row.numel() >= rows, "bigram_embedding rows")
+    buckets = pairs.shape[0] - 1
+    _need(table.is_contiguous() and pairs.is_contiguous() and table.dtype == pairs.dtype and pairs.shape[1] == width
+          and buckets >= 1, "bigram_embedding tables")
+    lib = load_library("hyper_streams")
+    # (multipliers modulo the buckets give the same rows and keep the products in 64 bits)
+    _check(lib.tb_bigram_embedding(_ptr(tokens), _ptr(positions), _ptr(seq_of_row), _ptr(row_start), _ptr(state_slots),
+                                   _ptr(table), _ptr(pairs), _ptr(before), _ptr(out), _i32(rows), _i32(width), _i32(copies),
+                                   _i32(table.shape[0]), _i32(buckets), _i64(mul_prev % buckets), _i64(mul_cur % buckets),
+                                   _i32(_code(table.dtype)), _stream()), "bigram_embedding")
+    return out
+
+
+# ----------------------------------------------------------------------------- recurrences over a matrix per head
+
+STATE_SPACE, MATRIX_MEMORY, DELTA_RULE = 0, 1, 2
+NORM_GATE_SIGMOID, NORM_GATE_SILU, NORM_GATE_SILU_FIRST = 0, 1, 2
+
+
+def matrix_state_shape(kind: int, heads: int, dim: int, vdim: int):
+    """The shape of a request's state: value columns (and the normaliser's, for the matrix memory) of ``dim`` numbers each,
+    rounded up to four."""
+    return (heads, vdim + (1 if kind == MATRIX_MEMORY else 0), -(-dim // 4) * 4)
+
+
+def matrix_recurrence(kind: int, rows: torch.Tensor, offsets, gates: torch.Tensor, per_head, state: torch.Tensor,
+                      out: torch.Tensor, row_start: torch.Tensor, state_slots: torch.Tensor, *, num_seqs: int, heads: int,
+                      qk_heads: int, dim: int, vdim: int, q_scale: float = 1.0, cap: float = 0.0,
+                      running: Optional[torch.Tensor] = None, aux: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``S_t = a_t S_(t-1) + k_t u_t^T``, ``o_t = q_scale S_t^T q_t`` per head over the step's rows of every sequence; ``offsets``: the
+    columns of ``rows`` at which q, k (``[qk_heads, dim]``) and v (``[heads, vdim]``) start; ``gates``: float32 logits.
+
+    ``STATE_SPACE``: ``dt = softplus(gates[h] + bias)``, ``a = exp(rate dt)``, ``u = dt v``, ``o += skip v``; ``per_head = (rate, bias, skip)``.
+    ``MATRIX_MEMORY``: log gates ``i = cap tanh((gates[h] + b_i) / cap)``, ``f = log sigmoid(cap tanh((gates[heads + h] + b_f) / cap))``,
+    ``m = max(f + m, i)`` (``running``, 0 at first), ``a = exp(f + m_before - m)``, ``u = exp(i - m) v``; ``per_head = (b_i, b_f)``; ``aux``
+    (float32 ``[T, heads, 2]``) receives the normaliser's ``n . q`` and ``m``.
+    ``DELTA_RULE``: unit q and k, ``a = exp(rate softplus(gates[h] + bias))``, ``u = sigmoid(gates[heads + h]) (v - a S^T k)``;
+    ``per_head = (rate, bias)``.
+
+    ``state``: float32 ``[slots, *matrix_state_shape(...)]``, read and renewed per sequence; ``out``: float32 ``[T, heads * vdim]``."""
+    _cuda(rows, gates, state, out, row_start, state_slots, running, aux, *per_head)
+    total = out.shape[0]
+    q_off, k_off, v_off = (int(o) for o in offsets)
+    reach = max(q_off + qk_heads * dim, k_off + qk_heads * dim, v_off + heads * vdim)
+    _need(rows.stride(1) == 1 and rows.shape[0] == total and rows.shape[1] >= reach and min(q_off, k_off, v_off) >= 0,
+          "matrix_recurrence rows")
+    want_gates = heads if kind == STATE_SPACE else 2 * heads
+    _need(gates.dtype == torch.float32 and gates.stride(1) == 1 and gates.shape[0] == total and gates.shape[1] >= want_gates,
+          "matrix_recurrence gates are float32 logits")
+    _f32_rows(out, (total, heads * vdim), "matrix_recurrence out is contiguous float32")
+    shape = matrix_state_shape(kind, heads, dim, vdim)
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == shape, "matrix_recurrence state")
+    vectors = list(per_head) + [None] * (3 - len(per_head))
+    _need(len(per_head) == (3 if kind == STATE_SPACE else 2), "matrix_recurrence vectors")
+    for v in per_head:
+        _f32_rows(v, (heads,), "matrix_recurrence vectors are float32 [heads]")
+    if kind == MATRIX_MEMORY:
+        _need(running is not None and running.dtype == torch.float32 and running.is_contiguous()
+              and tuple(running.shape[1:]) == shape[:2], "matrix_recurrence running maxima")
+        _need(aux is not None, "matrix_recurrence aux")
+        _f32_rows(aux, (total, heads, 2), "matrix_recurrence aux is float32 [rows, heads, 2]")
+    _need(row_start.dtype == torch.int32 and state_slots.dtype == torch.int32 and row_start.numel() > num_seqs
+          and state_slots.numel() >= num_seqs, "matrix_recurrence metadata must be int32")
+    lib = load_library("matrix_recurrence")
+    _check(lib.tb_matrix_recurrence(_i32(kind), _ptr(rows), _i64(rows.stride(0)), _i32(q_off), _i32(k_off), _i32(v_off),
+                                    _ptr(gates), _i64(gates.stride(0)), _ptr(vectors[0]), _ptr(vectors[1]), _ptr(vectors[2]),
+                                    _f32(cap), _f32(q_scale), _ptr(state), _ptr(running), _ptr(out), _ptr(aux),
+                                    _ptr(row_start), _ptr(state_slots), _i32(num_seqs), _i32(heads), _i32(qk_heads), _i32(dim),
+                                    _i32(vdim), _i32(_code(rows.dtype)), _stream()), "matrix_recurrence")
+    return out
+
+
+def recurrence_norm(v: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, groups: int, size: int,
+                    eps: float, gate_kind: int, aux: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out = rms(v) * weight * act(gate)`` over every run of ``size`` numbers of a row of float32 ``v`` (``NORM_GATE_SIGMOID``,
+    ``NORM_GATE_SILU``), or ``rms(v * silu(gate)) * weight`` (``NORM_GATE_SILU_FIRST``); ``weight`` holds ``size`` numbers for all runs
+    or ``groups * size``.  ``aux`` (see :func:`matrix_recurrence`): ``v`` is first divided by ``max(|n . q|, exp(-m)) + 1e-6``."""
+    _cuda(v, gate, weight, out, aux)
+    rows = v.shape[0]
+    _f32_rows(v, (rows, groups * size), "recurrence_norm takes contiguous float32 rows")
+    _f32_rows(aux, (rows, groups, 2), "recurrence_norm aux")
+    _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() in (size, groups * size), "recurrence_norm weight")
+    _need(gate.stride(1) == 1 and tuple(gate.shape) == (rows, groups * size) and out.stride(1) == 1
+          and tuple(out.shape) == (rows, groups * size) and out.dtype == gate.dtype, "recurrence_norm gate/out")
+    lib = load_library("matrix_recurrence")
+    _check(lib.tb_recurrence_norm(_ptr(v), _ptr(aux), _ptr(gate), _i64(gate.stride(0)), _ptr(weight), _i32(weight.numel()),
+                                  _ptr(out), _i64(out.stride(0)), _i32(rows), _i32(groups), _i32(size), _f32(eps),
+                                  _i32(gate_kind), _i32(_code(out.dtype)), _stream()), "recurrence_norm")
     return out

@@ -16,7 +16,7 @@ import torch
 
 from .. import kernels
 from ..config.spec import LayerSpec, ModelSpec, PartSpec
-from ..parts import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, INJECTIONS, MIXERS, NORMS, RESIDUAL_GATES, TOKEN_INPUTS, Block, CacheBinding, DeferredNorm,
+from ..parts import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, INJECTIONS, MIXERS, NORMS, RESIDUAL_GATES, STREAM_MIXINGS, TOKEN_INPUTS, Block, CacheBinding, DeferredNorm,
                      ResidualStream, Runtime, StepContext)
 from ..weights.loader import ExpectedTensor
 
@@ -43,6 +43,10 @@ def _part_specs(spec: ModelSpec):
             if not block_cls.accepts_residual_gates:
                 raise ValueError(f"block '{layer.block}' takes no residual gates")
             yield RESIDUAL_GATES, layer.residual_gates
+        if layer.stream_mixing is not None:
+            if not block_cls.accepts_stream_mixing:
+                raise ValueError(f"block '{layer.block}' takes no stream mixing")
+            yield STREAM_MIXINGS, layer.stream_mixing
     for injection in spec.injections:
         yield INJECTIONS, injection
     yield NORMS, spec.final_norm
@@ -96,6 +100,8 @@ class DecoderModel:
                 extras["token_input"] = build(TOKEN_INPUTS, layer.token_input)
             if layer.residual_gates is not None:
                 extras["residual_gates"] = build(RESIDUAL_GATES, layer.residual_gates)
+            if layer.stream_mixing is not None:
+                extras["stream_mixing"] = build(STREAM_MIXINGS, layer.stream_mixing)
             self.layers.append(block_cls(norms, mixer, feed_forward, **extras))
         self.injections = [build(INJECTIONS, part) for part in spec.injections]
         self.final_norm = build(NORMS, spec.final_norm)
@@ -106,7 +112,8 @@ class DecoderModel:
 
     # ------------------------------------------------------------------ cache description
     def cache_needs(self) -> List[Optional[object]]:
-        """For each run entry: its mixer's cache need, or ``None`` if it keeps no cache of its own."""
+        """For each run entry: its mixer's cache need, or ``None`` if it keeps no cache of its own; behind them, if the
+        embedding keeps something per request, its need (the embedding's binding is then the last one)."""
         needs: List[Optional[object]] = []
         for index, entry in enumerate(self.spec.run_order):
             need = self.layers[entry.layer].mixer.cache_need()
@@ -118,11 +125,20 @@ class DecoderModel:
                 needs.append(None)
             else:
                 needs.append(need)
-        return needs
+        own = self.embedding.cache_need()
+        return needs if own is None else needs + [own]
+
+    def cache_sources(self) -> List[Optional[int]]:
+        """For each of :meth:`cache_needs`: the earlier one whose cache it reads, or ``None``."""
+        sources = [entry.cache_of for entry in self.spec.run_order]
+        return sources if self.embedding.cache_need() is None else sources + [None]
 
     # ------------------------------------------------------------------ forward
-    def _embed(self, ctx: StepContext) -> torch.Tensor:
+    def _embed(self, ctx: StepContext, bindings: Sequence[Optional[CacheBinding]]) -> torch.Tensor:
         token_ids = ctx.token_ids[:ctx.num_rows]
+        if self.embedding.takes_context:
+            own = bindings[len(self.spec.run_order)] if self.embedding.cache_need() is not None else None
+            return self.embedding.forward(token_ids, ctx=ctx, cache=own)
         if self.embedding.takes_positions:
             return self.embedding.forward(token_ids, positions=ctx.positions[:ctx.num_rows])
         return self.embedding.forward(token_ids)
@@ -133,13 +149,14 @@ class DecoderModel:
         ``want_every_row``: the caller knows that ``want_rows`` is ``0 .. num_rows - 1`` (a decode step), so the
         rows need not be gathered before the head."""
         ctx.carried.clear()
-        hidden = self._embed(ctx)
+        hidden = self._embed(ctx, bindings)
         stream = ResidualStream(hidden, None)
         order = self.spec.run_order
         # the embedding output that injections read: rows of their own, since blocks add into the stream in place
         origin = None
         if any(injection.reads_origin for injection in self.injections):
-            origin = self._embed(ctx)
+            # (an embedding with a state of its own runs once a step)
+            origin = hidden.clone() if self.embedding.takes_context else self._embed(ctx, bindings)
         wants_logits = want_rows is not None and want_rows.numel() > 0
         every_row = wants_logits and want_every_row and want_rows.numel() == ctx.num_rows
         for index, entry in enumerate(order):

@@ -24,13 +24,16 @@ Kinds and what each must provide:
     arranges norms, mixer and feed-forward: ``forward(stream, ctx, cache)`` on a
     :class:`ResidualStream`.
 ``Embedding`` / ``Head``
-    ``forward(token_ids)`` (``forward(token_ids, positions=...)`` if it says ``takes_positions``) -> ``[T, hidden]`` /
+    ``forward(token_ids)`` (``forward(token_ids, positions=...)`` if it says ``takes_positions``, ``forward(token_ids, ctx=...,
+    cache=...)`` if it says ``takes_context``, with ``cache_need()`` like a mixer's for what it keeps per request) -> ``[T, hidden]`` /
     ``forward(x)`` -> float32 ``[S, vocab]``.
 ``Injection``
     ``forward(stream, origin, ctx)`` -> the new :class:`ResidualStream`: a step between two blocks that mixes the
     stream with the embedding output.
 ``TokenInput``
     ``forward(residual, ctx)``: a term a layer adds to the 32-bit stream behind its sublayers, from the step's tokens.
+``StreamMixing``
+    for a stream kept as several copies: per sublayer ``mix(which)`` and ``share(which)``, how the copies meet and take a result in.
 
 Every class also has ``expected_tensors(spec)`` -> ``{checkpoint name: ExpectedTensor}``
 so that the loader can check a checkpoint, and the random-weights writer can make one,
@@ -480,6 +483,11 @@ class FeedForward(Part):
 
 class Embedding(Part):
     takes_positions = False      # True if ``forward`` also takes ``positions`` (int32, one per token)
+    # True if ``forward`` takes the step (``ctx``) and the embedding's own cache binding (``cache``); it runs once a step
+    takes_context = False
+
+    def cache_need(self):
+        return None
 
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
@@ -520,6 +528,17 @@ class ResidualGates(Part):
         raise NotImplementedError
 
 
+class StreamMixing(Part):
+    """How the copies of a multi-copy stream meet around a sublayer (``"mixer"``, ``"feed_forward"``): ``mix(which)`` (float32
+    ``[copies, copies]``, from, to) and ``share(which)`` (float32 ``[copies]``, each copy's share of the sublayer's result)."""
+
+    def mix(self, which: str) -> torch.Tensor:
+        raise NotImplementedError
+
+    def share(self, which: str) -> torch.Tensor:
+        raise NotImplementedError
+
+
 class Head(Part):
     accepts_deferred_norm = False
 
@@ -537,6 +556,8 @@ class Block:
     accepts_token_input = False
     # True if the constructor takes ``residual_gates`` (a :class:`ResidualGates`)
     accepts_residual_gates = False
+    # True if the constructor takes ``stream_mixing`` (a :class:`StreamMixing`)
+    accepts_stream_mixing = False
 
     def __init__(self, norms: Mapping[str, Norm], mixer: Mixer, feed_forward: Optional[FeedForward]):
         self.norms = dict(norms)
@@ -566,3 +587,4 @@ HEADS: Registry[Head] = Registry("head")
 INJECTIONS: Registry[Injection] = Registry("injection")
 TOKEN_INPUTS: Registry[TokenInput] = Registry("token input")
 RESIDUAL_GATES: Registry[ResidualGates] = Registry("residual gates")
+STREAM_MIXINGS: Registry[StreamMixing] = Registry("stream mixing")

@@ -42,6 +42,15 @@ by feature, by a learned scale and by a gate that reads the sublayer's own input
 
 The weighting, the addition and the norm in front of the next sublayer (the next block's first norm, or the final norm)
 are one kernel (``gated_add_norm``); the gate's product leaves 32-bit logits.
+
+``hyper_connected`` is the pre-norm arrangement over a stream kept as several 32-bit copies ``x_1 .. x_s``:
+
+    h  = input_norm(copies);       x_t <- sum_s mix_1[s, t] x_s + out_1[t] mixer(h)
+    m  = post_mixer_norm(copies);  x_t <- sum_s mix_2[s, t] x_s + out_2[t] feed_forward(m)       (absent without one)
+
+whose norms read a weighted sum of the copies (``mixed_streams_rms_norm``).  The mixing, the taking in of the sublayer's result
+(of both results of two mixers side by side, with their weights) and the norm in front of the next sublayer (the next
+block's first norm, or the final norm) are one kernel (``mixed_streams_norm``).
 """
 
 from __future__ import annotations
@@ -277,6 +286,72 @@ class GatedPreNormBlock(Block):
                 rows = self.norms["post_mixer"].forward(residual)
             update = self.feed_forward.forward(rows, ctx)
             rows = self._join(residual, update, rows, "feed_forward", next_norm)
+        if rows is not None:
+            return ResidualStream(residual, None, prepared=FinishedNorm(next_norm, residual, rows))
+        return ResidualStream(residual, None)
+
+
+@BLOCKS.register("hyper_connected")
+class HyperConnectedBlock(Block):
+    """Norm roles ``input`` and, with a feed-forward, ``post_mixer``: norms over the copies of the stream that offer
+    ``stream_statistic()``; ``stream_mixing`` holds how the copies meet around each sublayer."""
+
+    accepts_next_norm = True
+    accepts_stream_mixing = True
+
+    def __init__(self, norms, mixer, feed_forward, stream_mixing=None):
+        super().__init__(norms, mixer, feed_forward)
+        if stream_mixing is None:
+            raise ValueError("a hyper_connected block needs its stream mixing")
+        self.mixing = stream_mixing
+        for role, norm in self.norms.items():
+            if not hasattr(norm, "stream_statistic") or norm.streams != stream_mixing.streams:
+                raise ValueError(f"a hyper_connected block takes norms over the stream's {stream_mixing.streams} copies; "
+                                 f"'{norm.kind}' ({role}) is not one")
+
+    @classmethod
+    def norm_roles(cls, with_feed_forward: bool = True) -> Tuple[str, ...]:
+        return ("input", "post_mixer") if with_feed_forward else ("input",)
+
+    def entry_norm(self) -> Optional[Norm]:
+        return self.norms["input"]
+
+    def _join(self, residual, update, which: str, following: Optional[Norm]):
+        """The copies mixed and ``update`` taken in, in place; the rows of ``following`` over the new copies, or None."""
+        import torch
+
+        from .. import kernels
+
+        statistic = getattr(following, "stream_statistic", lambda: None)() if following is not None else None
+        take = weight = out = None
+        eps = 0.0
+        if statistic is not None:
+            take, weight, eps = statistic
+            out = torch.empty((residual.shape[0], following.size), dtype=following.runtime.dtype, device=residual.device)
+        kernels.mixed_streams_norm(residual, update, self.mixing.mix(which), self.mixing.share(which), take, weight, out,
+                                   self.mixing.streams, eps)
+        return out
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, cache, next_norm: Optional[Norm] = None) -> ResidualStream:
+        import torch
+
+        residual = stream.residual
+        if stream.update is not None or stream.update_b is not None or residual.dtype != torch.float32:
+            raise NotImplementedError("a hyper_connected block takes the stream's 32-bit copies without a pending update")
+        if stream.prepared is not None and stream.prepared.norm is self.norms["input"]:
+            h = stream.prepared.materialize()
+        else:
+            h = self.norms["input"].forward(residual)
+        if hasattr(self.mixer, "forward_sides"):          # two results that are added with a weight each: by the joining kernel
+            (left, right), (left_scale, right_scale) = self.mixer.forward_sides(h, ctx, cache)
+            mixed = (left, left_scale, right, right_scale)
+        else:
+            mixed = (self.mixer.forward(h, ctx, cache), 1.0, None, 0.0)
+        last = self.feed_forward is None
+        rows = self._join(residual, mixed, "mixer", next_norm if last else self.norms["post_mixer"])
+        if not last:
+            update = self.feed_forward.forward(rows, ctx)
+            rows = self._join(residual, (update, 1.0, None, 0.0), "feed_forward", next_norm)
         if rows is not None:
             return ResidualStream(residual, None, prepared=FinishedNorm(next_norm, residual, rows))
         return ResidualStream(residual, None)

@@ -14,7 +14,7 @@ import torch
 from .. import kernels
 from ..config.spec import PartSpec
 from ..weights.loader import ExpectedTensor
-from .base import EMBEDDINGS, HEADS, Embedding, Head, Runtime
+from .base import EMBEDDINGS, HEADS, Embedding, Head, Runtime, StateNeed
 from .linear import BestOfRows, Linear
 
 
@@ -96,6 +96,53 @@ class PositionedEmbedding(Embedding):
         if out is None:
             out = torch.empty((token_ids.numel(), self.hidden_size), dtype=torch.float32, device=self.table.device)
         return kernels.embedding_norm(token_ids, positions, self.table, self.positions, self.weight, self.groups, self.eps, out)
+
+
+@EMBEDDINGS.register("bigram_embedding")
+class BigramEmbedding(Embedding):
+    """A token's row plus a row for the pair it forms with the token in front: ``table[token] + pairs[(token in front * mul_prev +
+    token * mul_cur) mod buckets]``, or the last row of ``pairs`` for a sequence's first token.  The rows come out in 32-bit,
+    ``copies`` times side by side (a stream kept as several copies starts with equal ones).
+
+    params: ``vocab_size, hidden_size, buckets, mul_prev, mul_cur``, optional ``copies``; weights: ``table``, ``pairs``
+    ``[buckets + 1, hidden]``.  A request's last token is state in its slot: a step's first token of a request pairs with it."""
+
+    graph_safe = True
+    takes_context = True
+
+    def __init__(self, spec: PartSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
+        super().__init__(spec, tensors, runtime)
+        p = spec.params
+        self.hidden_size = int(p["hidden_size"])
+        self.buckets = int(p["buckets"])
+        self.mul_prev, self.mul_cur = int(p["mul_prev"]), int(p["mul_cur"])
+        self.copies = int(p.get("copies") or 1)
+        if self.buckets < 1 or self.copies < 1:
+            raise ValueError("bigram_embedding needs at least one bucket and one copy")
+        self.table = runtime.matrix(tensors["table"])
+        self.pairs = runtime.matrix(tensors["pairs"])
+
+    @classmethod
+    def expected_tensors(cls, spec: PartSpec) -> Dict[str, ExpectedTensor]:
+        p, w = spec.params, spec.weights
+        hidden = int(p["hidden_size"])
+        return {w["table"]: ExpectedTensor((int(p["vocab_size"]), hidden)),
+                w["pairs"]: ExpectedTensor((int(p["buckets"]) + 1, hidden))}
+
+    @classmethod
+    def random_tensor(cls, spec, role, shape, generator) -> torch.Tensor:
+        return torch.randn(shape, generator=generator, dtype=torch.float32) * (0.5 if role == "pairs" else 1.0)
+
+    def cache_need(self) -> StateNeed:
+        return StateNeed((1,), torch.int32)
+
+    def forward(self, token_ids: torch.Tensor, ctx, cache, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if cache is None or cache.storage is None:
+            raise RuntimeError("bigram_embedding needs a state binding")
+        if out is None:
+            out = torch.empty((token_ids.numel(), self.copies * self.hidden_size), dtype=torch.float32, device=self.table.device)
+        return kernels.bigram_embedding(token_ids, ctx.positions, ctx.seq_of_row, ctx.row_start, ctx.state_slots, self.table,
+                                        self.pairs, cache.storage, out, self.copies, self.mul_prev, self.mul_cur)
 
 
 @HEADS.register("lm_head")

@@ -121,6 +121,53 @@ class GroupedRMSNorm(Norm):
         return kernels.group_rms_norm(residual, update, self.weight, self.groups, self.eps, self._out(residual, out))
 
 
+@NORMS.register("mixed_streams_rms_norm")
+class MixedStreamsRMSNorm(Norm):
+    """RMS norm of a weighted sum of the copies of a stream kept as ``streams`` 32-bit copies side by side:
+    ``u = sum_s take[s] x_s``, ``u / sqrt(mean(u^2) + eps) * weight``.
+
+    params: ``size`` (of one copy), ``streams``, ``eps``; weights: ``weight`` ``[size]`` and, unless every copy counts once,
+    ``take`` ``[streams]``.  The stream is float32 ``[T, streams * size]``; the normed rows ``[T, size]`` come out in the run
+    dtype, rounded once."""
+
+    graph_safe = True
+
+    def __init__(self, spec: PartSpec, tensors: Mapping[str, torch.Tensor], runtime: Runtime):
+        super().__init__(spec, tensors, runtime)
+        params = spec.params
+        self.size, self.streams, self.eps = int(params["size"]), int(params["streams"]), float(params["eps"])
+        if self.streams < 1:
+            raise ValueError("a stream has at least one copy")
+        self.weight = runtime.vector_f32(tensors["weight"])
+        if "take" in tensors:
+            self.take = runtime.vector_f32(tensors["take"])
+        else:
+            self.take = torch.ones(self.streams, dtype=torch.float32, device=runtime.device)
+
+    @classmethod
+    def expected_tensors(cls, spec: PartSpec) -> Dict[str, ExpectedTensor]:
+        p, w = spec.params, spec.weights
+        out = {w["weight"]: ExpectedTensor((int(p["size"]),))}
+        if "take" in w:
+            out[w["take"]] = ExpectedTensor((int(p["streams"]),))
+        return out
+
+    @classmethod
+    def random_tensor(cls, spec, role, shape: Tuple[int, ...], generator) -> torch.Tensor:
+        noise = torch.randn(shape, generator=generator, dtype=torch.float32)
+        return 1.0 / int(spec.params["streams"]) + noise * 0.2 if role == "take" else 1.0 + noise * 0.1
+
+    def stream_statistic(self):
+        """``(take, weight, eps)``: what the kernel that mixes the copies in front needs to take this norm as well."""
+        return self.take, self.weight, self.eps
+
+    def forward(self, x: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if out is None:
+            out = torch.empty((x.shape[0], self.size), dtype=self.runtime.dtype, device=x.device)
+        kernels.mixed_streams_norm(x, None, None, None, self.take, self.weight, out, self.streams, self.eps)
+        return out
+
+
 @NORMS.register("layer_norm")
 class LayerNorm(Norm):
     """Layer norm with weight and bias over a residual stream kept in 32-bit: ``(x - mean) / sqrt(var + eps) * weight +

@@ -7,8 +7,12 @@ Per row ``h`` (the mixer's input):
 * the position encoding (``rotary_blend``, rotate-half layout) turns the first ``dims`` numbers of every query and
   key head; with ``qk_norm_eps`` every query and key head is then divided by ``sqrt(mean(head^2) + qk_norm_eps)``
   (no weight); rotated, normalised keys and the values go into the request's pages;
+* with ``projection_norm_eps`` the norm stands in front of the rotation and runs over the whole projection instead: all heads'
+  queries over their one root mean square, times a weight per number, and the keys likewise; with ``values_from_keys`` there
+  is no value projection and a token's values are its keys as projected, before norm and rotation;
 * every row attends over the keys its mask lets it see: ``causal`` (all up to its own position), ``window`` (its own
-  and the ``size - 1`` positions before it; older pages go back to the pool) or ``window_pooled``: the window and, for
+  and the ``size - 1`` positions before it; older pages go back to the pool), ``blocks`` (the positions are cut into consecutive
+  blocks of ``size`` from 0, and a row sees its own block up to itself) or ``window_pooled``: the window and, for
   every block of ``pool`` positions that ends in front of it (blocks are counted from position 0; block ``b`` is seen
   from position ``p`` if ``(b + 1) * pool <= p - size + 1``), one key and one value that are the averages of the block's
   keys and values as the pages hold them; so for up to ``pool - 1`` steps a token is visible neither by itself nor through
@@ -17,6 +21,7 @@ Per row ``h`` (the mixer's input):
   on seeing (their pages stay; older pages behind the window go back to the pool).  Scores ``(q . k) * scale``, with ``softcap`` then ``softcap * tanh(score / softcap)``, the softmax
   and the weights are 32-bit; with ``sink`` the denominator also holds ``exp`` of a learned number per query head; with
   ``distance_bias`` the score of the key ``n`` positions back loses ``w * ln(1 + r * n)``, two numbers per query head;
+* with ``head_gate`` a head's output is multiplied by the sigmoid of one number that a projection of ``h`` gives it;
 * with ``bias`` the three projections add a bias each, with ``output_bias`` the output projection does;
 * values may be mixed across layers: a part with ``value_mix`` ``"first"`` leaves its values in the step
   (``StepContext.carried``), a later one with ``"mix"`` stores ``(1 - x) v + x v_first`` instead of its own values ``v``, ``x``
@@ -41,15 +46,18 @@ from .base import (MIXERS, POSITION_ENCODINGS, DeferredNorm, Mixer, PagedKeyValu
                    StepContext)
 from .linear import Linear
 
-_MASKS = {"causal": kernels.MASK_CAUSAL, "window": kernels.MASK_WINDOW, "window_pooled": kernels.MASK_WINDOW_POOLED}
+_MASKS = {"causal": kernels.MASK_CAUSAL, "window": kernels.MASK_WINDOW, "window_pooled": kernels.MASK_WINDOW_POOLED,
+          "blocks": kernels.MASK_BLOCKS}
 
 
 @MIXERS.register("normed_attention")
 class NormedAttention(Mixer):
     """params: ``hidden_size, num_heads, num_kv_heads, key_dim, value_dim, scale``, ``mask`` (``{"kind": "causal" |
-    "window" | "window_pooled", "size": n, "pool": P, "keep_first": k}``), ``qk_norm_eps`` (None: queries and keys stay as
+    "window" | "blocks" | "window_pooled", "size": n, "pool": P, "keep_first": k}``), ``qk_norm_eps`` (None: queries and keys stay as
     rotated), optional ``softcap``, ``sink`` (bool), ``bias`` (bool), ``output_bias`` (bool), ``distance_bias`` (bool),
-    ``value_mix`` (``"first"`` | ``"mix"``), ``stream``.  weights: ``q, k, v, o``, with ``bias`` also ``q_bias, k_bias,
+    ``value_mix`` (``"first"`` | ``"mix"``), ``projection_norm_eps``, ``values_from_keys`` (bool), ``head_gate`` (bool), ``stream``.  weights:
+    ``q, k, v, o`` (no ``v`` with ``values_from_keys``), with ``projection_norm_eps`` ``q_norm`` and ``k_norm`` (as wide as the
+    projections), with ``head_gate`` ``g`` ``[num_heads, hidden]``, with ``bias`` also ``q_bias, k_bias,
     v_bias``, with ``output_bias`` ``o_bias``, with ``sink`` ``sink`` ``[num_heads]``, with ``distance_bias`` ``distance_weight``
     and ``distance_rate`` (``[num_heads]`` each), to mix ``value_mix`` (one number).  children: ``position``."""
 
@@ -94,6 +102,20 @@ class NormedAttention(Mixer):
         eps = p.get("qk_norm_eps")
         self.unit_norm = eps is not None
         self.qk_norm_eps = float(eps) if eps is not None else 0.0
+        eps = p.get("projection_norm_eps")
+        self.projection_norm_eps = float(eps) if eps is not None else None
+        self.values_from_keys = bool(p.get("values_from_keys"))
+        self.projection_norm = None
+        if self.projection_norm_eps is not None:
+            if self.biased or self.unit_norm or self.value_mix is not None:
+                raise ValueError("a norm over the whole projection goes with no biases, no unit norm and no mixed values")
+            self.projection_norm = torch.cat([tensors["q_norm"], tensors["k_norm"]]).to(
+                device=runtime.device, dtype=torch.float32).contiguous()
+        elif self.values_from_keys:
+            raise ValueError("keys that are values come with a norm over the whole projection")
+        if self.values_from_keys and self.key_dim != self.value_dim:
+            raise ValueError("keys that are values have the values' width")
+        self.head_gated = bool(p.get("head_gate"))
         self.stream_f32 = p.get("stream") == "float32"
         if self.num_heads % self.num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
@@ -106,7 +128,14 @@ class NormedAttention(Mixer):
         if self.biased:
             self.in_bias = torch.cat([tensors["q_bias"], tensors["k_bias"], tensors["v_bias"]]).to(
                 device=runtime.device, dtype=torch.float32).contiguous()
-        self.in_proj = Linear(torch.cat([tensors["q"], tensors["k"], tensors["v"]], dim=0), runtime)
+        wide = [tensors["q"], tensors["k"]] + ([] if self.values_from_keys else [tensors["v"]])
+        self.gate_offset = sum(t.shape[0] for t in wide)
+        if self.head_gated:
+            wide.append(tensors["g"])
+            missing = -(self.gate_offset + self.num_heads) % 8      # (rows of zeros, so that projected rows start on 16 bytes)
+            if missing:
+                wide.append(torch.zeros((missing, self.hidden_size), dtype=tensors["g"].dtype))
+        self.in_proj = Linear(torch.cat(wide, dim=0), runtime)
         self.o_proj = Linear(tensors["o"], runtime, bias=tensors["o_bias"] if p.get("output_bias") else None)
         position_spec = spec.children.get("position") or PartSpec.make("none")
         self.position = POSITION_ENCODINGS.get(position_spec.kind)(position_spec, {}, runtime)
@@ -126,9 +155,14 @@ class NormedAttention(Mixer):
         out = {
             w["q"]: ExpectedTensor((heads * d, hidden)),
             w["k"]: ExpectedTensor((kv * d, hidden)),
-            w["v"]: ExpectedTensor((kv * dv, hidden)),
             w["o"]: ExpectedTensor((hidden, heads * dv)),
         }
+        if not p.get("values_from_keys"):
+            out[w["v"]] = ExpectedTensor((kv * dv, hidden))
+        if p.get("projection_norm_eps") is not None:
+            out.update({w["q_norm"]: ExpectedTensor((heads * d,)), w["k_norm"]: ExpectedTensor((kv * d,))})
+        if p.get("head_gate"):
+            out[w["g"]] = ExpectedTensor((heads, hidden))
         if p.get("bias"):
             out.update({w["q_bias"]: ExpectedTensor((heads * d,)), w["k_bias"]: ExpectedTensor((kv * d,)),
                         w["v_bias"]: ExpectedTensor((kv * dv,))})
@@ -148,6 +182,8 @@ class NormedAttention(Mixer):
             return torch.randn(shape, generator=generator, dtype=torch.float32) * 0.3
         if role in ("distance_weight", "distance_rate", "value_mix"):
             return torch.rand(shape, generator=generator, dtype=torch.float32) * 0.5 + 0.1
+        if role.endswith("_norm"):
+            return 1.0 + torch.randn(shape, generator=generator, dtype=torch.float32) * 0.1
         if role == "sink":
             return torch.randn(shape, generator=generator, dtype=torch.float32)
         return torch.randn(shape, generator=generator, dtype=torch.float32) * (shape[-1] ** -0.5)
@@ -156,7 +192,8 @@ class NormedAttention(Mixer):
         """``(name, Linear, epilogue)`` of the mixer's matrix products, for the printed kernel plan."""
         from .. import plan
 
-        return [("q/k/v", self.in_proj, plan.BF16), ("o", self.o_proj, plan.F32 if self.stream_f32 else plan.BF16)]
+        name = "q/k" + ("" if self.values_from_keys else "/v") + ("/gate" if self.head_gated else "")
+        return [(name, self.in_proj, plan.BF16), ("o", self.o_proj, plan.F32 if self.stream_f32 else plan.BF16)]
 
     def cache_need(self):
         if self.mask_kind == "window_pooled":
@@ -166,7 +203,8 @@ class NormedAttention(Mixer):
                     PooledBlocksNeed(num_kv_heads=self.num_kv_heads, key_dim=self.key_dim, value_dim=self.value_dim,
                                      pool=self.pool))
         return PagedKeyValueNeed(num_kv_heads=self.num_kv_heads, key_dim=self.key_dim, value_dim=self.value_dim,
-                                 window=self.mask_size if self.mask_kind == "window" else None, keep_first=self.keep_first)
+                                 window=self.mask_size if self.mask_kind == "window" else None,
+                                 block=self.mask_size if self.mask_kind == "blocks" else None, keep_first=self.keep_first)
 
     def attention_choice(self, rows: int) -> str:
         """The attention kernel of a step of ``rows`` rows (all three know the cap, the learned sink and pooled blocks)."""
@@ -199,13 +237,21 @@ class NormedAttention(Mixer):
             if first is None or first.shape != (rows, self.num_kv_heads * self.value_dim):
                 raise RuntimeError("a mixer that mixes values needs an earlier layer's values of the same width in the step")
             across["mix_values"] = (first, self.mix)
-        kernels.rope_norm_cache(proj, q, cache.storage, ctx.positions, ctx.seq_of_row, group.block_table, self.inv_freq,
-                                amplitude=self.amplitude, heads=self.num_heads, kv_heads=self.num_kv_heads,
-                                dim=self.key_dim, vdim=self.value_dim, rot_dims=self.rot_dims,
-                                unit_norm=self.unit_norm, eps=self.qk_norm_eps, page_size=cache.page_size,
-                                bias=self.in_bias, **across)
+        if self.projection_norm is not None:
+            kernels.row_norm_rope_cache(proj, q, cache.storage, ctx.positions, ctx.seq_of_row, group.block_table, self.inv_freq,
+                                        self.projection_norm, amplitude=self.amplitude, heads=self.num_heads,
+                                        kv_heads=self.num_kv_heads, dim=self.key_dim, vdim=self.value_dim,
+                                        rot_dims=self.rot_dims, eps=self.projection_norm_eps, page_size=cache.page_size,
+                                        values_from_keys=self.values_from_keys)
+        else:
+            kernels.rope_norm_cache(proj, q, cache.storage, ctx.positions, ctx.seq_of_row, group.block_table, self.inv_freq,
+                                    amplitude=self.amplitude, heads=self.num_heads, kv_heads=self.num_kv_heads,
+                                    dim=self.key_dim, vdim=self.value_dim, rot_dims=self.rot_dims,
+                                    unit_norm=self.unit_norm, eps=self.qk_norm_eps, page_size=cache.page_size,
+                                    bias=self.in_bias, **across)
         extras = {"sinks": self.sinks, "softcap": self.softcap, "keep_first": self.keep_first,
-                  "distance_bias": self.distance_bias}
+                  "distance_bias": self.distance_bias,
+                  "head_gate": proj[:, self.gate_offset:self.gate_offset + self.num_heads] if self.head_gated else None}
         if pooled is not None:
             pool_table = ctx.groups[pooled.group].block_table
             kernels.pool_blocks(cache.storage, pooled.storage, ctx.positions, ctx.seq_of_row, group.block_table, pool_table,

@@ -75,7 +75,9 @@ class ParallelMixers(Mixer):
         needs = tuple(n for part in self.sides for n in _needs_of(part.cache_need()))
         return needs if needs else None
 
-    def forward(self, x, ctx: StepContext, cache):
+    def forward_sides(self, x, ctx: StepContext, cache):
+        """``((left rows, right rows), (left_scale, right_scale))``: the two results (32-bit) before they are added, for a block
+        whose own kernel adds them."""
         if isinstance(x, DeferredNorm):
             x = x.materialize()
         bindings = tuple(cache) if isinstance(cache, tuple) else (() if cache is None else (cache,))
@@ -89,4 +91,8 @@ class ParallelMixers(Mixer):
         left, right = results
         if left.dtype != torch.float32 or right.dtype != torch.float32:
             raise NotImplementedError("parallel_mixers adds 32-bit rows (its mixers leave them for a 32-bit stream)")
-        return kernels.blend_rows(left, right, self.scales[0], self.scales[1])
+        return (left, right), self.scales
+
+    def forward(self, x, ctx: StepContext, cache):
+        (left, right), (left_scale, right_scale) = self.forward_sides(x, ctx, cache)
+        return kernels.blend_rows(left, right, left_scale, right_scale)
