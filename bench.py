@@ -664,7 +664,7 @@ def run_kernels(args):
 
 
 # ----------------------------------------------------------------------------- another design beside Llama
-# `--design revesun|pekodra|kazodra|ladedra|rirulix`: prefill and decode of a model of that design at layer sizes like a real model's (random
+# `--design revesun|pekodra|kazodra|ladedra|rirulix|tibivik`: prefill and decode of a model of that design at layer sizes like a real model's (random
 # weights), beside a Llama (and, for Pekodra, a Revesun: the other design with a 32-bit stream) of the same width, heads, head sizes, layer count and about as many weights a layer, measured the
 # same way; then the design's own kernels alone, against the bytes they must move.  The default workload is untouched.
 DESIGN_SIZES = {
@@ -827,6 +827,46 @@ def rirulix_config(size, layers):
             "layers": [dict(recurrent if i % 2 else attention, mlp=moe) for i in range(layers)]}
 
 
+TIBIVIK_SIZES = {
+    # (attention sides have the heads of the models beside it; state-space layers are twice as wide as the stream; both recurrences of
+    # the two-sided layers have Ladedra's retention heads; the middle `looped` of the `stored` layers is walked twice)
+    "1b": dict(window=512, chunk=512, rot_dims=32, space_heads=64, space_dim=64, state=128, groups=1, heads=16, dim=128, taps=4, streams=4,
+               dense_ff=8192, stored=10, looped=(2, 8)),
+    "3b": dict(window=512, chunk=512, rot_dims=64, space_heads=96, space_dim=64, state=128, groups=1, heads=24, dim=128, taps=4, streams=4,
+               dense_ff=8192, stored=8, looped=(2, 6)),
+    "8b": dict(window=512, chunk=512, rot_dims=64, space_heads=128, space_dim=64, state=128, groups=8, heads=32, dim=128, taps=4, streams=4,
+               dense_ff=14336, stored=5, looped=(1, 4)),
+}
+
+
+def tibivik_config(size, layers):
+    """State-space layers in turn with layers of two mixers: chunked attention beside the gated delta rule, and window attention
+    beside a matrix memory; dense feed-forwards; a stream of four copies; a run in the middle is walked twice, so that `layers`
+    layer runs happen in all (as many as the models beside it run)."""
+    z, p = DESIGN_SIZES[size], TIBIVIK_SIZES[size]
+    stored, (start, stop) = p["stored"], p["looped"]
+    if layers != z["layers"]:
+        stored, start, stop = layers, 0, 0
+    space = {"type": "mamba2", "mixer": {"heads": p["space_heads"], "vdim": p["space_dim"], "state": p["state"], "groups": p["groups"],
+                                         "norm_groups": p["groups"], "conv": p["taps"]}}
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5}
+    chunked = {"type": "parallel_2", "mixer": {
+        "left": dict(left, mask={"size": p["chunk"]}),
+        "right": {"heads": p["heads"], "kv_heads": p["heads"] // 2, "dim": p["dim"], "vdim": p["dim"], "conv": p["taps"]},
+        "left_scale": 1.0, "right_scale": 1.0}}
+    windowed = {"type": "parallel", "mixer": {
+        "left": dict(left, mask={"size": p["window"]}, rot={"dims": p["rot_dims"], "base": 500000.0}),
+        "right": {"heads": p["heads"], "dim": p["dim"], "vdim": p["dim"], "gate_cap": 15.0}, "left_scale": 1.0, "right_scale": 1.0}}
+    dense = {"kind": "dense", "ff": p["dense_ff"]}
+    order = [space, chunked, space, windowed]
+    config = {"architecture": "Tibivik", "torch_dtype": "bfloat16", "width": z["width"], "vocab": DESIGN_VOCAB, "streams": p["streams"],
+              "norm": {"eps": 1e-5}, "embedding": {"bigram": {"buckets": 65536, "mul_prev": 31, "mul_cur": 7}},
+              "layers": [dict(order[i % 4], mlp=dense) for i in range(stored)]}
+    if stop > start:
+        config["loop"] = {"start": start, "stop": stop, "times": 2}
+    return config
+
+
 def run_design(args):
     import numpy as np
     import torch
@@ -910,7 +950,7 @@ def run_design(args):
         return out
 
     result = {"design": {"revesun": "Revesun", "pekodra": "Pekodra", "kazodra": "Kazodra", "ladedra": "Ladedra",
-                         "rirulix": "Rirulix"}[args.design],
+                         "rirulix": "Rirulix", "tibivik": "Tibivik"}[args.design],
               "size": args.size,
               "layers": layers,
               "vocab": DESIGN_VOCAB, "dtype": "bf16", "data": "synthetic",
@@ -945,6 +985,17 @@ def run_design(args):
             result["llama"] = measure(llama)
         if args.only in ("all", "kernels"):
             result["kernels"] = rirulix_kernels(args.size, pk)
+        result["clocks"] = sampler.stop(windows)
+        result["peaks"] = pk
+        print(json.dumps(result))
+        return 0
+    if args.design == "tibivik":                   # beside Ladedra: two mixers side by side, a matrix state, a 32-bit stream
+        if args.only in ("all", "decode", "prefill"):
+            result["tibivik"] = measure(tibivik_config(args.size, layers))
+            result["ladedra"] = measure(ladedra_config(args.size, layers))
+            result["llama"] = measure(llama)
+        if args.only in ("all", "kernels"):
+            result["kernels"] = tibivik_kernels(args.size, pk)
         result["clocks"] = sampler.stop(windows)
         result["peaks"] = pk
         print(json.dumps(result))
@@ -1690,6 +1741,182 @@ def rirulix_kernels(size, pk):
     return out
 
 
+def tibivik_kernels(size, pk):
+    """Tibivik's own kernels alone at this size, timed like :func:`design_kernels`, each behind the like kernel of another
+    model of the package at the same size ("beside: ..."): 2,048 prompt rows of one sequence, and 64 and 8 decoded rows at
+    context 2,048."""
+    import torch
+
+    from tesseract_b200 import kernels
+
+    z, p = DESIGN_SIZES[size], TIBIVIK_SIZES[size]
+    dev, bf16 = "cuda", torch.bfloat16
+    W, page, copies = z["width"], PAGE_SIZE, p["streams"]
+    H, G, d = z["heads"], z["kv_heads"], z["dim"]
+    SH, sd, N, groups, taps = p["space_heads"], p["space_dim"], p["state"], p["groups"], p["taps"]
+    RH, rd, rot = p["heads"], p["dim"], p["rot_dims"]
+    half_freq = torch.tensor([5e5 ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=torch.float32, device=dev)
+    full_freq = torch.tensor([5e5 ** (-2.0 * i / d) for i in range(d // 2)], dtype=torch.float32, device=dev)
+    sinks = torch.randn(H, device=dev)
+    out = {}
+
+    def timed(name, make, nbytes, flops=0, tensor=False):
+        time_launches(pk, out, name, make, nbytes, flops, tensor)
+
+    def rows_of(rows, width, dtype=bf16):
+        return torch.randn(rows, width, device=dev).to(dtype)
+
+    for label, rows, seqs, begin in (("prefill_2048", 2048, 1, 0), ("decode_64", 64, 64, 2047), ("decode_8", 8, 8, 2047)):
+        new = rows // seqs
+        positions = (torch.arange(rows, dtype=torch.int32, device=dev) % new) + begin
+        seq_of_row = torch.arange(rows, dtype=torch.int32, device=dev) // new
+        row_start = torch.arange(seqs + 1, dtype=torch.int32, device=dev) * new
+        seq_begin = torch.full((seqs,), begin, dtype=torch.int32, device=dev)
+        slots = torch.arange(seqs, dtype=torch.int32, device=dev)
+        pages_per_seq = 2048 // page
+        table = (torch.arange(seqs * pages_per_seq, dtype=torch.int32, device=dev) + 1).view(seqs, pages_per_seq)
+        page_elems = G * page * 2 * d
+        new_pages = lambda: torch.randn(seqs * pages_per_seq + 1, page_elems, device=dev).to(bf16)
+
+        def embed(k):
+            tokens = torch.randint(0, DESIGN_VOCAB, (rows,), dtype=torch.int32, device=dev)
+            tab, pairs = rows_of(DESIGN_VOCAB, W), rows_of(4097, W)
+            before, y = torch.zeros(seqs + 1, 1, dtype=torch.int32, device=dev), torch.empty(rows, copies * W, device=dev)
+            return lambda: kernels.bigram_embedding(tokens, positions, seq_of_row, row_start, slots, tab, pairs, before, y, copies, 31, 7)
+
+        timed(f"bigram_embedding (4 copies)/{label}", embed, rows * W * (2 + 2 + 4 * copies))
+
+        def join(both):
+            def make(k):
+                res, a, b = rows_of(rows, copies * W, torch.float32), rows_of(rows, W, torch.float32), rows_of(rows, W, torch.float32)
+                mix, share, take = torch.eye(copies, device=dev), torch.ones(copies, device=dev), torch.full((copies,), 0.25, device=dev)
+                w, y = torch.ones(W, device=dev), torch.empty(rows, W, dtype=bf16, device=dev)
+                update = (a, 1.0, b, 1.0) if both else (a, 1.0, None, 0.0)
+                return lambda: kernels.mixed_streams_norm(res, update, mix, share, take, w, y, copies, 1e-5)
+            return make
+
+        timed(f"mixed_streams_norm (4 copies, two results)/{label}", join(True), rows * W * (4 * (2 * copies + 2) + 2))
+        timed(f"mixed_streams_norm (4 copies, one result)/{label}", join(False), rows * W * (4 * (2 * copies + 1) + 2))
+
+        def gated_join(k):
+            res, upd, gate = (rows_of(rows, W, torch.float32) for _ in range(3))
+            bias, scale, w = torch.zeros(W, device=dev), torch.ones(W, device=dev), torch.ones(W, device=dev)
+            y = torch.empty(rows, W, dtype=bf16, device=dev)
+            return lambda: kernels.gated_add_norm(res, upd, gate, bias, scale, w, y, 1e-5)
+
+        timed(f"beside: gated_add_norm (Ladedra)/{label}", gated_join, rows * W * (4 * 4 + 2))
+
+        def row_norm(k):
+            proj, q, cache = rows_of(rows, (H + G) * d), torch.empty(rows, H * d, dtype=bf16, device=dev), new_pages()
+            w = torch.ones((H + G) * d, device=dev)
+            return lambda: kernels.row_norm_rope_cache(proj, q, cache, positions, seq_of_row, table, half_freq, w, amplitude=1.0, heads=H,
+                                                       kv_heads=G, dim=d, vdim=d, rot_dims=rot, eps=1e-5, page_size=page,
+                                                       values_from_keys=True)
+
+        timed(f"row_norm_rope_cache (keys are values)/{label}", row_norm, rows * d * 2 * ((H + G) + H + 2 * G))
+
+        def rotate(k):
+            proj, q, cache = rows_of(rows, (H + 2 * G) * d), torch.empty(rows, H * d, dtype=bf16, device=dev), new_pages()
+            return lambda: kernels.rope_norm_cache(proj, q, cache, positions, seq_of_row, table, full_freq, amplitude=1.0, heads=H,
+                                                   kv_heads=G, dim=d, vdim=d, rot_dims=d, unit_norm=True, eps=1e-5, page_size=page)
+
+        timed(f"beside: rope_norm_cache (Ladedra)/{label}", rotate, rows * (H + 2 * G) * d * 4)
+
+        def attend(kernel, mask, size, extras):
+            def make(k):
+                q, y, cache = rows_of(rows, H * d), torch.empty(rows, H * d, dtype=bf16, device=dev), new_pages()
+                common = dict(heads=H, kv_heads=G, dim=d, vdim=d, page_size=page, mask_kind=mask, mask_size=size, scale=d ** -0.5,
+                              **extras(k))
+                if kernel == "prompt":
+                    return lambda: kernels.attention_prompt_mma(q, y, cache, positions, row_start, table, num_seqs=seqs, **common)
+                return lambda: kernels.attention_rows_mma(q, y, cache, positions, seq_of_row, table, **common)
+            return make
+
+        kind = "prompt" if rows > 256 else "rows"
+        window, chunk = p["window"], p["chunk"]
+        for what, mask, size, extras, seen in (
+                (f"window {window}, sink", kernels.MASK_WINDOW, window, lambda k: {"sinks": sinks},
+                 [min(window, int(t) + 1) for t in positions.tolist()]),
+                (f"chunks of {chunk}, sink, gate per head", kernels.MASK_BLOCKS, chunk,
+                 lambda k: {"sinks": sinks, "head_gate": rows_of(rows, H)}, [int(t) % chunk + 1 for t in positions.tolist()]),
+                ("beside: plain window", kernels.MASK_WINDOW, window, lambda k: {}, [min(window, int(t) + 1) for t in positions.tolist()])):
+            moved = rows * H * d * 4 + (sum(seen) if new == 1 else rows) * 2 * G * d * 2
+            name = f"attention_{kind}_mma"
+            timed(f"beside: {name} (window {window}, Pekodra)/{label}" if what.startswith("beside") else f"{name} ({what})/{label}",
+                  attend(kind, mask, size, extras), moved, sum(seen) * H * d * 4, True)
+
+        channels = SH * sd + 2 * groups * N
+
+        def conv(k):
+            proj, u = rows_of(rows, SH * sd + channels), torch.empty(rows, channels, dtype=bf16, device=dev)
+            w, b = torch.randn(taps, channels, device=dev), torch.randn(channels, device=dev)
+            state = torch.zeros(seqs + 1, taps - 1, channels, device=dev)
+            return lambda: kernels.short_conv(proj[:, SH * sd:], None, w, b, state, u, positions, seq_of_row, row_start, seq_begin, slots,
+                                              num_seqs=seqs, single=new == 1, activation=True)
+
+        def conv_beside(k):
+            proj, u = rows_of(rows, SH * sd + channels), torch.empty(rows, channels, dtype=bf16, device=dev)
+            w, b = torch.randn(taps, channels, device=dev), torch.randn(channels, device=dev)
+            state = torch.zeros(seqs + 1, taps - 1, channels, device=dev)
+            return lambda: kernels.short_conv(proj[:, SH * sd:], b, w, b, state, u, positions, seq_of_row, row_start, seq_begin, slots,
+                                              num_seqs=seqs, single=new == 1)
+
+        moved = rows * channels * 4 + seqs * (taps - 1) * channels * (8 if new == 1 else 4)
+        timed(f"short_conv (SiLU, with its state)/{label}", conv, moved)
+        timed(f"beside: short_conv (Rirulix)/{label}", conv_beside, moved)
+
+        def recur(code, heads, qk, dim, vdim, gates_a_head, vectors):
+            def make(k):
+                x = rows_of(rows, 2 * qk * dim + heads * vdim)
+                gates = rows_of(rows, gates_a_head * heads, torch.float32)
+                per_head = [-torch.rand(heads, device=dev) for _ in range(vectors)]
+                shape = kernels.matrix_state_shape(code, heads, dim, vdim)
+                state, y = torch.zeros(seqs + 1, *shape, device=dev), torch.empty(rows, heads * vdim, device=dev)
+                more = {}
+                if code == kernels.MATRIX_MEMORY:
+                    more = dict(running=torch.zeros(seqs + 1, *shape[:2], device=dev), aux=torch.empty(rows, heads, 2, device=dev), cap=15.0)
+                return lambda: kernels.matrix_recurrence(code, x, (0, qk * dim, 2 * qk * dim), gates, per_head, state, y, row_start, slots,
+                                                         num_seqs=seqs, heads=heads, qk_heads=qk, dim=dim, vdim=vdim, max_new=new, q_scale=0.1, **more)
+            return make
+
+        for name, code, heads, qk, dim, vdim, gates_a_head, vectors, per in (
+                ("state space", kernels.STATE_SPACE, SH, groups, N, sd, 1, 3, 4), ("matrix memory", kernels.MATRIX_MEMORY, RH, RH, rd, rd, 2, 2, 4),
+                ("delta rule", kernels.DELTA_RULE, RH, RH // 2, rd, rd, 2, 2, 6)):
+            timed(f"matrix_recurrence ({name})/{label}", recur(code, heads, qk, dim, vdim, gates_a_head, vectors),
+                  rows * ((2 * qk * dim + heads * vdim) * 2 + heads * vdim * 4 + gates_a_head * heads * 4) + seqs * heads * dim * vdim * 8,
+                  flops=rows * heads * dim * vdim * per)
+
+        def retention(heads, dim, vdim):
+            def make(k):
+                x, decay = rows_of(rows, heads * (2 * dim + vdim), torch.float32), torch.full((heads,), 0.99, device=dev)
+                state, y = torch.zeros(seqs + 1, heads, dim, vdim, device=dev), torch.empty(rows, heads * vdim, device=dev)
+                return lambda: kernels.lightning(x, decay, state, y, row_start, slots, num_seqs=seqs, heads=heads, dim=dim, vdim=vdim,
+                                                 max_new=new, activation=False)
+            return make
+
+        for heads, dim, vdim in ((RH, rd, rd), (SH, N, sd)):
+            timed(f"beside: lightning ({heads} heads of {dim} by {vdim}, Ladedra)/{label}", retention(heads, dim, vdim),
+                  rows * heads * (2 * dim + 2 * vdim) * 4 + seqs * heads * dim * vdim * 8, flops=rows * heads * dim * vdim * 4)
+
+        def norm(parts, part, gate_kind, aux):
+            def make(k):
+                v, gate, y = rows_of(rows, parts * part, torch.float32), rows_of(rows, parts * part), torch.empty(rows, parts * part, dtype=bf16, device=dev)
+                w, a = torch.ones(parts * part, device=dev), torch.randn(rows, parts, 2, device=dev) if aux else None
+                return lambda: kernels.recurrence_norm(v, gate, w, y, groups=parts, size=part, eps=1e-5, gate_kind=gate_kind, aux=a)
+            return make
+
+        timed(f"recurrence_norm (state space)/{label}", norm(groups, SH * sd // groups, kernels.NORM_GATE_SILU_FIRST, False), rows * SH * sd * 8)
+        timed(f"recurrence_norm (matrix memory)/{label}", norm(RH, rd, kernels.NORM_GATE_SIGMOID, True), rows * RH * rd * 8)
+        timed(f"recurrence_norm (delta rule)/{label}", norm(RH, rd, kernels.NORM_GATE_SILU, False), rows * RH * rd * 8)
+
+        def head_norm(k):
+            o, gate, y = rows_of(rows, RH * rd, torch.float32), rows_of(rows, RH * rd), torch.empty(rows, RH * rd, dtype=bf16, device=dev)
+            return lambda: kernels.head_norm_gate(o, gate, y, heads=RH, vdim=rd, eps=1e-5, gate_kind=kernels.GATE_SILU)
+
+        timed(f"beside: head_norm_gate (Ladedra)/{label}", head_norm, rows * RH * rd * 8)
+    return out
+
+
 def pekodra_kernels(size, pk):
     """Pekodra's own kernels alone at this size, timed like :func:`design_kernels`: 2,048 prompt rows of one sequence,
     and 64 decoded rows at context 2,048."""
@@ -1892,7 +2119,7 @@ def main():
     parser.add_argument("--workload", choices=["3b", "8b"], default=None,
                         help="run another workload instead of the headline one: continuous batching at the 3B sizes, "
                              "or a 2,048-token portion beside 64 decode rows at the 8B sizes")
-    parser.add_argument("--design", choices=["revesun", "pekodra", "kazodra", "ladedra", "rirulix"], default=None,
+    parser.add_argument("--design", choices=["revesun", "pekodra", "kazodra", "ladedra", "rirulix", "tibivik"], default=None,
                         help="instead of the headline workload: prefill and decode of this design beside a Llama of "
                              "equal layer sizes (--size), and the design's own kernels alone")
     args = parser.parse_args()

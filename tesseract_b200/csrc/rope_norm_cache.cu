@@ -258,9 +258,21 @@ row_norm_rope_cache_kernel(const T* __restrict__ proj, int64_t proj_stride, T* _
         cosines[i] = cs * g.amplitude;
         sines[i] = sn * g.amplitude;
     }
-    const float inv_q = 1.0f / sqrtf(block_sum(qq, scratch) / (float)q_width + g.eps);
-    const float inv_k = 1.0f / sqrtf(block_sum(kk, scratch) / (float)(both - q_width) + g.eps);
-    __syncthreads();
+    qq = warp_sum(qq);
+    kk = warp_sum(kk);
+    if ((threadIdx.x & 31) == 0) {
+        scratch[threadIdx.x >> 5] = qq;
+        scratch[kRowThreads / 32 + (threadIdx.x >> 5)] = kk;
+    }
+    __syncthreads();                                   // (the row, its sines and cosines and the warps' sums are there)
+    qq = kk = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kRowThreads / 32; ++w) {
+        qq += scratch[w];
+        kk += scratch[kRowThreads / 32 + w];
+    }
+    const float inv_q = 1.0f / sqrtf(qq / (float)q_width + g.eps);
+    const float inv_k = 1.0f / sqrtf(kk / (float)(both - q_width) + g.eps);
     const int page = block_table[(int64_t)seq_of_row[row] * bt_stride + pos / g.page_size], in_page = pos % g.page_size;
     T* keys = cache + (int64_t)page * g.kv_heads * g.page_size * (g.dim + g.vdim);
     T* values = keys + (int64_t)g.kv_heads * g.page_size * g.dim;

@@ -18,7 +18,12 @@
 
 namespace {
 
-__device__ __forceinline__ float activated(float y, int act) { return act ? y / (1.0f + expf(-y)) : y; }
+// SiLU: accurate for 32-bit outputs; in front of a rounding to bfloat16 with the fast exponential and division
+template <typename T>
+__device__ __forceinline__ float activated(float y, int act) {
+    if (!act) return y;
+    return sizeof(T) == 4 ? y / (1.0f + expf(-y)) : __fdividef(y, 1.0f + __expf(-y));
+}
 
 // A thread a (row, channel): any width, any number of taps.
 template <typename T, bool SINGLE>
@@ -47,7 +52,7 @@ short_conv_kernel(const T* __restrict__ proj, int64_t proj_stride, const float* 
         if (SINGLE && j > 0) st[(int64_t)(j - 1) * channels] = v;      // (index j - 1 has been read: the walk ascends)
     }
     if (out_bias != nullptr) sum += out_bias[c];
-    Elem<T>::store(out + (int64_t)row * out_stride + c, activated(sum, act));
+    Elem<T>::store(out + (int64_t)row * out_stride + c, activated<T>(sum, act));
 }
 
 template <int N>
@@ -141,7 +146,7 @@ short_conv_packets_kernel(const T* __restrict__ proj, int64_t proj_stride, const
             float sum = 0.0f;
 #pragma unroll
             for (int j = 0; j < J; ++j) sum = fmaf(w[j][e], v[j][e], sum);
-            y[e] = activated(sum + behind[e], act);
+            y[e] = activated<T>(sum + behind[e], act);
         }
         if (SINGLE) {
 #pragma unroll

@@ -1804,7 +1804,7 @@ def matrix_state_shape(kind: int, heads: int, dim: int, vdim: int):
 
 def matrix_recurrence(kind: int, rows: torch.Tensor, offsets, gates: torch.Tensor, per_head, state: torch.Tensor,
                       out: torch.Tensor, row_start: torch.Tensor, state_slots: torch.Tensor, *, num_seqs: int, heads: int,
-                      qk_heads: int, dim: int, vdim: int, q_scale: float = 1.0, cap: float = 0.0,
+                      qk_heads: int, dim: int, vdim: int, max_new: int, q_scale: float = 1.0, cap: float = 0.0,
                       running: Optional[torch.Tensor] = None, aux: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``S_t = a_t S_(t-1) + k_t u_t^T``, ``o_t = q_scale S_t^T q_t`` per head over the step's rows of every sequence; ``offsets``: the
     columns of ``rows`` at which q, k (``[qk_heads, dim]``) and v (``[heads, vdim]``) start; ``gates``: float32 logits.
@@ -1816,7 +1816,8 @@ def matrix_recurrence(kind: int, rows: torch.Tensor, offsets, gates: torch.Tenso
     ``DELTA_RULE``: unit q and k, ``a = exp(rate softplus(gates[h] + bias))``, ``u = sigmoid(gates[heads + h]) (v - a S^T k)``;
     ``per_head = (rate, bias)``.
 
-    ``state``: float32 ``[slots, *matrix_state_shape(...)]``, read and renewed per sequence; ``out``: float32 ``[T, heads * vdim]``."""
+    ``state``: float32 ``[slots, *matrix_state_shape(...)]``, read and renewed per sequence; ``out``: float32 ``[T, heads * vdim]``;
+    ``max_new``: the most rows any sequence brings."""
     _cuda(rows, gates, state, out, row_start, state_slots, running, aux, *per_head)
     total = out.shape[0]
     q_off, k_off, v_off = (int(o) for o in offsets)
@@ -1845,7 +1846,8 @@ def matrix_recurrence(kind: int, rows: torch.Tensor, offsets, gates: torch.Tenso
                                     _ptr(gates), _i64(gates.stride(0)), _ptr(vectors[0]), _ptr(vectors[1]), _ptr(vectors[2]),
                                     _f32(cap), _f32(q_scale), _ptr(state), _ptr(running), _ptr(out), _ptr(aux),
                                     _ptr(row_start), _ptr(state_slots), _i32(num_seqs), _i32(heads), _i32(qk_heads), _i32(dim),
-                                    _i32(vdim), _i32(_code(rows.dtype)), _stream()), "matrix_recurrence")
+                                    _i32(vdim), _i32(1 if max_new == 1 else 0), _i32(_code(rows.dtype)), _stream()),
+           "matrix_recurrence")
     return out
 
 

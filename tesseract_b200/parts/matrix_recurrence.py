@@ -96,7 +96,7 @@ class _MatrixMixer(Mixer):
         out = torch.empty((rows.shape[0], self.o_width), dtype=torch.float32, device=rows.device)
         return kernels.matrix_recurrence(self.recurrence, rows, offsets, gates, per_head, state, out, ctx.row_start,
                                          ctx.state_slots, num_seqs=ctx.num_seqs, heads=self.num_heads, qk_heads=qk_heads,
-                                         dim=self.key_dim, vdim=self.value_dim, **more)
+                                         dim=self.key_dim, vdim=self.value_dim, max_new=ctx.max_new, **more)
 
     def _finish(self, v, gate, *, groups: int, size: int, gate_kind: int, aux=None) -> torch.Tensor:
         normed = torch.empty((v.shape[0], self.o_width), dtype=gate.dtype, device=gate.device)

@@ -91,6 +91,8 @@ def portions_of(cut, T):
         return [(0, 10)] + [(p, p + 1) for p in range(10, T)]
     if cut == "twos":
         return [(p, min(p + 2, T)) for p in range(0, T, 2)]
+    if cut == "groups":
+        return [(p, min(p + 20, T)) for p in range(0, T, 20)]
     edges = list(range(0, T, 37)) + [T]
     return list(zip(edges[:-1], edges[1:]))
 
@@ -257,8 +259,9 @@ def test_recurrences_in_portions_and_batches_over_used_slots(dtype, kind, m):
 
 
 @pytest.mark.parametrize("kind,m", [c for c in CASES if c[1].get("conv", 4) > 1])
-def test_a_cut_of_the_recurrence_changes_no_bit(kind, m):
-    """The recurrence kernel itself, in 32-bit: a row's result depends on the state and on the row alone."""
+def test_cuts_of_the_recurrence_differ_by_rounding(kind, m):
+    """The recurrence kernel itself on 32-bit rows: groups of rows begin where a portion begins, and single rows take a kernel of
+    their own; results and states agree to a few roundings, and cuts at multiples of a group bit for bit."""
     from tesseract_b200 import kernels
 
     codes = {"state_space": kernels.STATE_SPACE, "matrix_memory": kernels.MATRIX_MEMORY, "gated_delta": kernels.DELTA_RULE}
@@ -276,16 +279,20 @@ def test_a_cut_of_the_recurrence_changes_no_bit(kind, m):
         out, aux = torch.empty(T, heads * vdim, device=dev()), torch.zeros(T, heads, 2, device=dev())
         for lo, hi in portions_of(cut, T):
             kernels.matrix_recurrence(code, rows[lo:hi], (0, qk * dim, 2 * qk * dim), gates[lo:hi], vectors, state, out[lo:hi], i32([0, hi - lo]),
-                                      i32([1]), num_seqs=1, heads=heads, qk_heads=qk, dim=dim, vdim=vdim, q_scale=0.3, cap=5.0,
+                                      i32([1]), num_seqs=1, heads=heads, qk_heads=qk, dim=dim, vdim=vdim, max_new=hi - lo, q_scale=0.3, cap=5.0,
                                       running=running if kind == "matrix_memory" else None,
                                       aux=aux[lo:hi] if kind == "matrix_memory" else None)
         return out, aux, state
 
     first = run("prompt")
     assert not first[2][0].any(), "a slot of another request was touched"
-    for cut in ("decode", "twos", "portions"):
+    for cut in ("decode", "twos", "portions", "groups"):
         for one, other in zip(first, run(cut)):
-            assert torch.equal(one, other), cut
+            assert torch.isfinite(other).all()
+            if cut == "groups":
+                assert torch.equal(one, other)
+            else:
+                assert float((one - other).abs().max()) <= 2e-5 * max(1.0, float(one.abs().max())), cut
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
