@@ -36,6 +36,8 @@
 namespace {
 
 enum Kind : int { STATE_SPACE = 0, MEMORY = 1, DELTA = 2 };
+constexpr int kWorkers = 8;          // the most warps that hold state
+constexpr int kFewBlocks = 120;      // fewer blocks than this leave multiprocessors idle
 constexpr int kProducers = 4;        // warps that prepare the next tile of rows
 
 typedef unsigned long long pair32;   // two neighbouring 32-bit floats
@@ -84,6 +86,15 @@ __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
 }
 
+__device__ __forceinline__ float widen(float v) { return v; }
+__device__ __forceinline__ float widen(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T narrow(float v);
+template <>
+__device__ __forceinline__ float narrow<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 narrow<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
 struct Recurrence {
     int64_t stride;                  // elements between rows of q, k and v
     int q_off, k_off, v_off;
@@ -99,17 +110,20 @@ struct Recurrence {
     int heads, qk_heads, dim, vdim, columns, workers, tile;
 };
 
-// The logits of a row's head -> (decay, write weight), for MEMORY (log f, log i) instead.
+// A row's gate logits of one head, and (decay, write weight) from them; for MEMORY (log f, log i) instead.
 template <int KIND>
-__device__ __forceinline__ float2 gates_of(const Recurrence& p, int row, int head, float rate, float bias0, float bias1) {
+__device__ __forceinline__ float2 logits_of(const Recurrence& p, int row, int head) {
     const float* gate = p.gates + (int64_t)row * p.gate_stride;
+    return make_float2(gate[head], KIND == STATE_SPACE ? 0.0f : gate[p.heads + head]);
+}
+template <int KIND>
+__device__ __forceinline__ float2 gates_of(float2 logits, float cap, float rate, float bias0, float bias1) {
     if (KIND == STATE_SPACE) {
-        const float dt = softplus(gate[head] + bias0);
+        const float dt = softplus(logits.x + bias0);
         return make_float2(expf(rate * dt), dt);
     }
-    const float first = gate[head], second = gate[p.heads + head];
-    if (KIND == DELTA) return make_float2(expf(rate * softplus(first + bias0)), 1.0f / (1.0f + expf(-second)));
-    return make_float2(log_sigmoid(p.cap * tanhf((second + bias1) / p.cap)), p.cap * tanhf((first + bias0) / p.cap));
+    if (KIND == DELTA) return make_float2(expf(rate * softplus(logits.x + bias0)), 1.0f / (1.0f + expf(-logits.y)));
+    return make_float2(log_sigmoid(cap * tanhf((logits.y + bias1) / cap)), cap * tanhf((logits.x + bias0) / cap));
 }
 
 // sum over the lanes of COUNT (a power of two up to 32) values: afterwards lane l holds the sum of value l % COUNT
@@ -131,13 +145,14 @@ __device__ __forceinline__ float spread_sums(float* v, int lane) {
 }
 
 constexpr int kGroup = 4;            // rows that share a pass over the state
+constexpr int kTile = 16;            // the most rows of a tile
 // a group's coefficients in shared memory: g_i iq_i [4], w_i or beta_i [4], p_3j ik_j [4], g_3 (and three unused), the triangle
 // iq_i p_ij ik_j (q_i . k_j) [4][4] and, for DELTA, beta_i ik_i g_i [4], the strict triangle beta_i ik_i p_ij ik_j (k_i . k_j) [8]
 template <int KIND>
 struct Coefficients { static constexpr int N = KIND == DELTA ? 44 : 32; };
 
 template <typename T, int KIND, int LPC, int NJ>
-__global__ void __launch_bounds__((4 + kProducers) * 32)
+__global__ void __launch_bounds__((kWorkers + kProducers) * 32)
 matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
     constexpr int DP = 4 * LPC * NJ;                 // numbers of q or k in shared memory (zeros behind dim)
     constexpr int CPL = 2, CW = 32 / LPC * CPL;
@@ -164,19 +179,21 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
         const float rate = KIND == MEMORY ? 0.0f : p.p0[head];
         const float bias0 = KIND == MEMORY ? p.p0[head] : p.p1[head], bias1 = KIND == MEMORY ? p.p1[head] : 0.0f;
         float m = KIND == MEMORY ? p.running[of_slot * p.columns + col0] : 0.0f;      // (the same in every producer)
-        float rq[kGroup][AHEAD ? E : 1], rk[kGroup][AHEAD ? E : 1], rv[kGroup];
+        // the next rows as they are stored: widened when they are used, so that nothing waits for them before
+        T rq[kGroup][AHEAD ? E : 1], rk[kGroup][AHEAD ? E : 1], rv[kGroup];
+        const T zero = narrow<T>(0.0f), one = narrow<T>(1.0f);
         const int groups = TT / kGroup;
         auto row_at = [&](int tile, int group, int t) { return first + tile * TT + group * kGroup + t; };
         auto there = [&](int tile, int group, int t) { return tile * TT + group * kGroup + t < n; };
         auto fetch_v = [&](int tile, int group, int t) {
             const int col = col0 + lane;
-            if (lane >= VC || !there(tile, group, t)) return 0.0f;
-            if (col < p.vdim) return Elem<T>::load(rows + (int64_t)row_at(tile, group, t) * p.stride + p.v_off + (int64_t)head * p.vdim + col);
-            return KIND == MEMORY && col == p.vdim ? 1.0f : 0.0f;
+            if (lane >= VC || !there(tile, group, t)) return zero;
+            if (col < p.vdim) return rows[(int64_t)row_at(tile, group, t) * p.stride + p.v_off + (int64_t)head * p.vdim + col];
+            return KIND == MEMORY && col == p.vdim ? one : zero;
         };
         auto fetch_qk = [&](int tile, int group, int t, int e, bool key) {
-            if (e >= p.dim || !there(tile, group, t)) return 0.0f;
-            return Elem<T>::load(rows + (int64_t)row_at(tile, group, t) * p.stride + (key ? p.k_off : p.q_off) + (int64_t)qk_head * p.dim + e);
+            if (e >= p.dim || !there(tile, group, t)) return zero;
+            return rows[(int64_t)row_at(tile, group, t) * p.stride + (key ? p.k_off : p.q_off) + (int64_t)qk_head * p.dim + e];
         };
         auto fetch = [&](int tile, int group) {
 #pragma unroll
@@ -191,25 +208,27 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
                 }
             }
         };
-        auto fetch_gates = [&](int tile) {            // a lane a row of the tile: decay and weight (1 and 0 behind the last row)
+        auto fetch_gates = [&](int tile) {            // a lane a row of the tile
             const int at = tile * TT + lane;
-            float2 g = make_float2(KIND == MEMORY ? 0.0f : 1.0f, 0.0f);
-            if (lane < TT && at < n) g = gates_of<KIND>(p, first + at, head, rate, bias0, bias1);
-            return g;
+            return lane < TT && at < n ? logits_of<KIND>(p, first + at, head) : make_float2(0.0f, 0.0f);
         };
-        float2 gate = fetch_gates(0);
+        float2 logits = fetch_gates(0);
         if (mine < groups) fetch(0, mine);
         for (int tile = -1; tile < tiles; ++tile) {
             const int next = tile + 1;
             if (next < tiles) {
                 float* buffer = smem + (next & 1) * stage;
                 float *qs = buffer, *ks = qs + TT * DP, *vs = ks + TT * DP, *cf = vs + TT * VC;
-                float a = gate.x, w = gate.y;
+                const int count = min(TT, n - next * TT);
+                const float2 gate = gates_of<KIND>(logits, p.cap, rate, bias0, bias1);
+                float a = lane < count ? gate.x : 1.0f, w = lane < count ? gate.y : 0.0f;    // (nothing happens behind the last row)
                 if (KIND == MEMORY) {
-                    const int count = min(TT, n - next * TT);
                     float before = 0.0f, now = 0.0f;
-                    for (int t = 0; t < count; ++t) {    // in token order
-                        const float f = __shfl_sync(0xffffffffu, gate.x, t), i = __shfl_sync(0xffffffffu, gate.y, t);
+                    // in token order; behind the last row log f = 0 and log i = -inf leave m as it is
+                    const float log_f = lane < count ? gate.x : 0.0f, log_i = lane < count ? gate.y : -INFINITY;
+#pragma unroll
+                    for (int t = 0; t < kTile; ++t) {
+                        const float f = __shfl_sync(0xffffffffu, log_f, t), i = __shfl_sync(0xffffffffu, log_i, t);
                         const float to = fmaxf(f + m, i);
                         if (lane == t) { before = m; now = to; }
                         m = to;
@@ -244,7 +263,8 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
                     if constexpr (AHEAD) {
 #pragma unroll
                         for (int i = 0; i < E; ++i) {
-                            const float q[kGroup] = {rq[0][i], rq[1][i], rq[2][i], rq[3][i]}, k[kGroup] = {rk[0][i], rk[1][i], rk[2][i], rk[3][i]};
+                            const float q[kGroup] = {widen(rq[0][i]), widen(rq[1][i]), widen(rq[2][i]), widen(rq[3][i])};
+                            const float k[kGroup] = {widen(rk[0][i]), widen(rk[1][i]), widen(rk[2][i]), widen(rk[3][i])};
                             take(i, q, k);
                         }
                     } else {
@@ -253,15 +273,15 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
                             float q[kGroup], k[kGroup];
 #pragma unroll
                             for (int t = 0; t < kGroup; ++t) {
-                                q[t] = fetch_qk(next, group, t, i * 32 + lane, false);
-                                k[t] = fetch_qk(next, group, t, i * 32 + lane, true);
+                                q[t] = widen(fetch_qk(next, group, t, i * 32 + lane, false));
+                                k[t] = widen(fetch_qk(next, group, t, i * 32 + lane, true));
                             }
                             take(i, q, k);
                         }
                     }
                     if (lane < VC)
 #pragma unroll
-                        for (int t = 0; t < kGroup; ++t) vs[(t0 + t) * VC + lane] = rv[t];
+                        for (int t = 0; t < kGroup; ++t) vs[(t0 + t) * VC + lane] = widen(rv[t]);
                     const float dot = spread_sums<DOTS>(dots, lane);
                     // lane l: dot product l; its pair (i, j), and the decays between
                     float ga[kGroup], gw[kGroup];
@@ -317,7 +337,7 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
                     }
                 }
                 if (next + 1 < tiles) {                   // the next tile's rows, asked for while the consumers work
-                    gate = fetch_gates(next + 1);
+                    logits = fetch_gates(next + 1);
                     if (mine < groups) fetch(next + 1, mine);
                 }
             }
@@ -329,7 +349,9 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
     }
 
     // ---------------------------------------------------------------------- consumers: the state of this warp's columns
-    const int r = lane % LPC, wcol = warp * CW + lane / LPC * CPL;
+    // (neighbouring lanes share a packet of q and k and own different columns: a shared-memory read serves them together)
+    constexpr int LANES = 32 / LPC;
+    const int r = lane / LANES, wcol = warp * CW + lane % LANES * CPL;
     pair32 S[CPL][NJ][2];
 #pragma unroll
     for (int j = 0; j < CPL; ++j) {
@@ -423,18 +445,18 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
                     for (int i = 0; i < half; ++i) {
                         const bool upper = r & half;
                         const float keep = upper ? d[i + half] : d[i], give = upper ? d[i] : d[i + half];
-                        d[i] = keep + __shfl_xor_sync(0xffffffffu, give, half);
+                        d[i] = keep + __shfl_xor_sync(0xffffffffu, give, half * LANES);
                     }
                 float sum = d[0];
 #pragma unroll
-                for (int o = 8; o < LPC; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+                for (int o = 8; o < LPC; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o * LANES);
                 const float4 share = *reinterpret_cast<const float4*>(c + 32), n0 = *reinterpret_cast<const float4*>(c + 36);
                 const float2 n1 = *reinterpret_cast<const float2*>(c + 40);
 #pragma unroll
                 for (int j = 0; j < CPL; ++j) {
                     float k[kGroup];
 #pragma unroll
-                    for (int t = 0; t < kGroup; ++t) k[t] = __shfl_sync(0xffffffffu, sum, (lane & ~7) | (t * 2 + j));
+                    for (int t = 0; t < kGroup; ++t) k[t] = __shfl_sync(0xffffffffu, sum, lane % LANES + (t * 2 + j) * LANES);
                     u[0][j] = fmaf(-share.x, k[0], u[0][j]);
                     u[1][j] = fmaf(-n0.x, u[0][j], fmaf(-share.y, k[1], u[1][j]));
                     u[2][j] = fmaf(-n0.z, u[1][j], fmaf(-n0.y, u[0][j], fmaf(-share.z, k[2], u[2][j])));
@@ -471,11 +493,11 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
                 for (int i = 0; i < half; ++i) {
                     const bool upper = r & half;
                     const float keep = upper ? d[i + half] : d[i], give = upper ? d[i] : d[i + half];
-                    d[i] = keep + __shfl_xor_sync(0xffffffffu, give, half);
+                    d[i] = keep + __shfl_xor_sync(0xffffffffu, give, half * LANES);
                 }
             float sum = d[0];
 #pragma unroll
-            for (int o = 8; o < LPC; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            for (int o = 8; o < LPC; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o * LANES);
             const bool second = r & 1;
             const float4 inside = *reinterpret_cast<const float4*>(c + 16 + my_t * 4);
             float o = c[my_t] * sum;
@@ -558,7 +580,7 @@ matrix_recurrence_step_kernel(const T* __restrict__ rows, Recurrence p, int runs
     for (int j = 0; j < CPL; ++j)
         v[j] = col + j < p.vdim ? Elem<T>::load(x + p.v_off + (int64_t)head * p.vdim + col + j)
                                 : (KIND == MEMORY && col + j == p.vdim ? 1.0f : 0.0f);
-    float2 gate = gates_of<KIND>(p, row, head, rate, bias0, bias1);
+    const float2 gate = gates_of<KIND>(logits_of<KIND>(p, row, head), p.cap, rate, bias0, bias1);
     float a = gate.x, w = gate.y;
     if (KIND == MEMORY) {
         const float before = p.running[of_slot * p.columns + min(col, p.columns - 1)];     // (every column holds the same)
@@ -653,9 +675,9 @@ int launch_as(const void* rows, Recurrence p, int num_seqs, int single, cudaStre
         return launched == cudaSuccess ? tb_launch_status() : (int)launched;
     }
     // few blocks: fewer columns a block, so that more multiprocessors take part
-    p.workers = 4;
-    while (p.workers > 1 && (int64_t)num_seqs * p.heads * ((p.columns + p.workers * CW - 1) / (p.workers * CW)) < 120) p.workers /= 2;
-    p.tile = DP > 512 ? 8 : 16;
+    p.workers = min(kWorkers, 32 / CW);
+    while (p.workers > 1 && (int64_t)num_seqs * p.heads * ((p.columns + p.workers * CW - 1) / (p.workers * CW)) < kFewBlocks) p.workers /= 2;
+    p.tile = DP > 512 ? kTile / 2 : kTile;
     const int VC = p.workers * CW;
     const size_t smem = sizeof(float) * 2 * (p.tile * (2 * DP + VC) + p.tile / kGroup * Coefficients<KIND>::N);
     auto kernel = matrix_recurrence_kernel<T, KIND, LPC, NJ>;
@@ -675,9 +697,13 @@ int launch_kind(const void* rows, const Recurrence& p, int num_seqs, int single,
     if (packets <= 8) return launch_as<T, KIND, 8, 1>(rows, p, num_seqs, single, stream);
     if (packets <= 16) return launch_as<T, KIND, 8, 2>(rows, p, num_seqs, single, stream);
     if (packets <= 24) return launch_as<T, KIND, 8, 3>(rows, p, num_seqs, single, stream);
-    if (packets <= 32) return launch_as<T, KIND, 8, 4>(rows, p, num_seqs, single, stream);
-    if (packets <= 48) return launch_as<T, KIND, 8, 6>(rows, p, num_seqs, single, stream);
-    if (packets <= 64) return launch_as<T, KIND, 8, 8>(rows, p, num_seqs, single, stream);
+    if (packets <= 32) {
+        // (where whole blocks of 32 columns would leave multiprocessors idle, a column is shared by twice the lanes)
+        if (single || (int64_t)num_seqs * p.heads * ((p.columns + 31) / 32) >= kFewBlocks) return launch_as<T, KIND, 8, 4>(rows, p, num_seqs, single, stream);
+        return launch_as<T, KIND, 16, 2>(rows, p, num_seqs, single, stream);
+    }
+    if (packets <= 48) return launch_as<T, KIND, 16, 3>(rows, p, num_seqs, single, stream);
+    if (packets <= 64) return launch_as<T, KIND, 16, 4>(rows, p, num_seqs, single, stream);
     if (packets <= 128) return launch_as<T, KIND, 32, 4>(rows, p, num_seqs, single, stream);
     return launch_as<T, KIND, 32, 8>(rows, p, num_seqs, single, stream);
 }
@@ -855,7 +881,7 @@ TB_EXPORT int tb_matrix_recurrence(int kind, const void* rows, int64_t stride, i
     p.gates = gates; p.gate_stride = gate_stride; p.p0 = p0; p.p1 = p1; p.p2 = p2; p.cap = cap; p.q_scale = q_scale;
     p.state = state; p.running = running; p.out = out; p.aux = aux; p.row_start = row_start; p.state_slots = state_slots;
     p.heads = heads; p.qk_heads = qk_heads; p.dim = dim; p.vdim = vdim; p.columns = kind == MEMORY ? vdim + 1 : vdim;
-    p.workers = 4; p.tile = 16;
+    p.workers = 1; p.tile = kTile;
     if (dtype == TB_F32) return launch_dtype<float>(kind, rows, p, num_seqs, single, stream);
     if (dtype == TB_BF16) return launch_dtype<__nv_bfloat16>(kind, rows, p, num_seqs, single, stream);
     return TB_ERR_BAD_DTYPE;
