@@ -63,6 +63,9 @@ __device__ __forceinline__ pair32 mul2(pair32 a, pair32 b) {
 }
 
 __device__ __forceinline__ float softplus(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+// e^x of a decay: near 1 through expm1f, whose result rounds to the nearest number once more; the plain function's last bit leans
+// to one side there, which a state that remembers thousands of tokens adds up
+__device__ __forceinline__ float decay_of(float x) { return x > -0.5f ? 1.0f + expm1f(x) : expf(x); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 
 // four numbers in a row, widened / rounded
@@ -120,9 +123,9 @@ template <int KIND>
 __device__ __forceinline__ float2 gates_of(float2 logits, float cap, float rate, float bias0, float bias1) {
     if (KIND == STATE_SPACE) {
         const float dt = softplus(logits.x + bias0);
-        return make_float2(expf(rate * dt), dt);
+        return make_float2(decay_of(rate * dt), dt);
     }
-    if (KIND == DELTA) return make_float2(expf(rate * softplus(logits.x + bias0)), 1.0f / (1.0f + expf(-logits.y)));
+    if (KIND == DELTA) return make_float2(decay_of(rate * softplus(logits.x + bias0)), 1.0f / (1.0f + expf(-logits.y)));
     return make_float2(log_sigmoid(cap * tanhf((logits.y + bias1) / cap)), cap * tanhf((logits.x + bias0) / cap));
 }
 
@@ -233,7 +236,7 @@ matrix_recurrence_kernel(const T* __restrict__ rows, Recurrence p) {
                         if (lane == t) { before = m; now = to; }
                         m = to;
                     }
-                    a = lane < count ? expf(gate.x + before - now) : 1.0f;
+                    a = lane < count ? decay_of(gate.x + before - now) : 1.0f;
                     w = lane < count ? expf(gate.y - now) : 0.0f;
                     if (mine == 0 && lane < count && col0 <= p.vdim && p.vdim < col0 + VC)
                         p.aux[((int64_t)(first + next * TT + lane) * p.heads + head) * 2 + 1] = now;
@@ -585,7 +588,7 @@ matrix_recurrence_step_kernel(const T* __restrict__ rows, Recurrence p, int runs
     if (KIND == MEMORY) {
         const float before = p.running[of_slot * p.columns + min(col, p.columns - 1)];     // (every column holds the same)
         const float now = fmaxf(gate.x + before, gate.y);
-        a = expf(gate.x + before - now);
+        a = decay_of(gate.x + before - now);
         w = expf(gate.y - now);
         __syncwarp();
         if (r == 0) {
