@@ -239,24 +239,45 @@ row_norm_rope_cache_kernel(const T* __restrict__ proj, int64_t proj_stride, T* _
     const int q_width = g.heads * g.dim, both = q_width + g.kv_heads * g.dim, half = g.rot_dims >> 1;
     float *cosines = row_smem + both, *sines = cosines + half;
     const T* prow = proj + (int64_t)row * proj_stride;
+    // everything that comes from memory is asked for before the sines and cosines are taken: the thread's first numbers and
+    // their weights, and the row's page
+    auto load = [&](int i, float* v, float* w) {
+        if constexpr (VEC) {
+            Packet<T>::load(prow + i, v);
+#pragma unroll
+            for (int e = 0; e < N; e += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(weight + i + e);
+                w[e] = f.x; w[e + 1] = f.y; w[e + 2] = f.z; w[e + 3] = f.w;
+            }
+        } else {
+            v[0] = Elem<T>::load(prow + i);
+            w[0] = weight[i];
+        }
+    };
     float qq = 0.0f, kk = 0.0f;
-    for (int i = threadIdx.x * N; i < both; i += kRowThreads * N) {
-        float v[N];
-        if constexpr (VEC) Packet<T>::load(prow + i, v);
-        else v[0] = Elem<T>::load(prow + i);
+    auto take = [&](int i, const float* v, const float* w) {
         float sum = 0.0f;
 #pragma unroll
         for (int e = 0; e < N; ++e) {
-            row_smem[i + e] = v[e];
+            row_smem[i + e] = v[e] * w[e];             // (the root mean square divides later)
             sum = fmaf(v[e], v[e], sum);
         }
         if (i < q_width) qq += sum; else kk += sum;    // (a packet does not straddle: widths are multiples of a head)
-    }
+    };
+    const int i0 = threadIdx.x * N;
+    float v0[N], w0[N];
+    if (i0 < both) load(i0, v0, w0);
+    const int page = block_table[(int64_t)seq_of_row[row] * bt_stride + pos / g.page_size], in_page = pos % g.page_size;
     for (int i = threadIdx.x; i < half; i += kRowThreads) {
         float sn, cs;
         sincosf((float)pos * inv_freq[i], &sn, &cs);
         cosines[i] = cs * g.amplitude;
         sines[i] = sn * g.amplitude;
+    }
+    if (i0 < both) take(i0, v0, w0);
+    for (int i = i0 + kRowThreads * N; i < both; i += kRowThreads * N) {
+        load(i, v0, w0);
+        take(i, v0, w0);
     }
     qq = warp_sum(qq);
     kk = warp_sum(kk);
@@ -273,7 +294,6 @@ row_norm_rope_cache_kernel(const T* __restrict__ proj, int64_t proj_stride, T* _
     }
     const float inv_q = 1.0f / sqrtf(qq / (float)q_width + g.eps);
     const float inv_k = 1.0f / sqrtf(kk / (float)(both - q_width) + g.eps);
-    const int page = block_table[(int64_t)seq_of_row[row] * bt_stride + pos / g.page_size], in_page = pos % g.page_size;
     T* keys = cache + (int64_t)page * g.kv_heads * g.page_size * (g.dim + g.vdim);
     T* values = keys + (int64_t)g.kv_heads * g.page_size * g.dim;
     for (int i = threadIdx.x * N; i < both; i += kRowThreads * N) {
@@ -282,13 +302,13 @@ row_norm_rope_cache_kernel(const T* __restrict__ proj, int64_t proj_stride, T* _
         const float inv = is_key ? inv_k : inv_q;
         float v[N];
 #pragma unroll
-        for (int e = 0; e < N; ++e) v[e] = row_smem[i + e] * inv * weight[i + e];
+        for (int e = 0; e < N; ++e) v[e] = row_smem[i + e] * inv;
         if (at < g.rot_dims) {                         // (with VEC a packet lies wholly in one half)
             const bool second = at >= half;
             const int other = second ? i - half : i + half, angle = second ? at - half : at;
 #pragma unroll
             for (int e = 0; e < N; ++e) {
-                const float w = row_smem[other + e] * inv * weight[other + e];
+                const float w = row_smem[other + e] * inv;
                 v[e] = second ? v[e] * cosines[angle + e] + w * sines[angle + e] : v[e] * cosines[angle + e] - w * sines[angle + e];
             }
         }
@@ -310,7 +330,7 @@ int launch_row_norm(const void* proj, int64_t proj_stride, void* q_out, int64_t 
                     const int* seq_of_row, const int* block_table, int bt_stride, const float* inv_freq, const float* weight,
                     int rows, const HeadGeometry& g, int values_from_keys, cudaStream_t stream) {
     constexpr int N = Packet<T>::N;
-    const uintptr_t bits = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache;
+    const uintptr_t bits = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache | (uintptr_t)weight;
     const bool vec = g.dim % N == 0 && g.vdim % N == 0 && (g.rot_dims / 2) % N == 0 && proj_stride % N == 0 && q_stride % N == 0 &&
                      bits % 16 == 0;
     const size_t smem = sizeof(float) * ((size_t)(g.heads + g.kv_heads) * g.dim + g.rot_dims);

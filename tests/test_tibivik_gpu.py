@@ -24,7 +24,7 @@ TOL = {torch.float32: 2e-5, torch.bfloat16: 3e-2}
 # In bfloat16 a result may also differ by this many times what rounding to bfloat16 alone moves in the plain computation
 # (``store=plain.bfloat16``): the package rounds at other places than the plain functions do, so the two are two draws of
 # that noise, and in these tiny models single positions amplify it.
-NOISE = 5.0
+NOISE = 4.0
 # In float32 a result may differ by this many times what rounding every weight to 32-bit once more moves in the plain model
 # (``reweighed``): tiny random models hold spots (a head whose output its own norm divides by almost nothing, say) that
 # amplify any rounding; a lost key, a stale state or a reach one off moves a logit by percents.
@@ -565,9 +565,9 @@ _PLAIN = {}
 
 
 def plain_rows(folder, requests, dtype):
-    """Per request the plain model's logits and what rounding alone (of what a bfloat16 run stores; of the weights to 32-bit)
-    moves in the plain model's logits of any of the requests."""
-    want, noise = {}, 0.0
+    """Per request the plain model's logits, and what rounding alone (of what a bfloat16 run stores; of the weights to 32-bit)
+    moves in the plain model's logits at the positions of all requests (the largest |difference| of each)."""
+    want, moved = {}, []
     config, tensors = plain.load_folder(folder)
     for rid, tokens in requests.items():
         key = (folder, tuple(tokens))
@@ -577,22 +577,30 @@ def plain_rows(folder, requests, dtype):
         if dtype not in noises:
             others = ([plain.forward(config, tensors, tokens, store=plain.bfloat16)[0]] if dtype == "bfloat16"
                       else [plain.forward(config, reweighed(tensors, seed), tokens)[0] for seed in range(3)])
-            noises[dtype] = max(float(np.abs(other - exact).max()) for other in others)
-        want[rid], noise = exact, max(noise, noises[dtype])
-    return want, noise
+            noises[dtype] = np.max([np.abs(other - exact).max(axis=1) for other in others], axis=0)
+        want[rid] = exact
+        moved.append(noises[dtype])
+    return want, np.concatenate(moved)
 
 
 def replay_against_plain(stepper, steps, folder, requests, dtype, what):
-    """Replay a trace and compare every wanted row with the plain model: ``REL`` of the request's largest |logit|, or what
-    rounding alone moves in the plain model, ``NOISE`` or ``NOISE_32`` times."""
-    want, noise = plain_rows(folder, requests, dtype)
+    """Replay a trace and compare every wanted row with the plain model.  No row may differ by more than ``REL`` of the
+    request's largest |logit| or ``NOISE`` (``NOISE_32``) times what rounding alone moves anywhere in the plain model, and of all rows
+    at most one in twenty by more than that many times what rounding moves at nine positions of ten."""
+    want, moved = plain_rows(folder, requests, dtype)
     got = replay(stepper, steps)
     assert got, f"{what}: nothing was replayed"
+    times = NOISE if dtype == "bfloat16" else NOISE_32
+    usual, over = float(np.quantile(moved, 0.9)), []
     for (rid, position), row in sorted(got.items(), key=lambda kv: (str(kv[0][0]), kv[0][1])):
-        limit = max(REL[dtype] * float(np.abs(want[rid]).max()), (NOISE if dtype == "bfloat16" else NOISE_32) * noise)
+        scale = float(np.abs(want[rid]).max())
+        limit = max(REL[dtype] * scale, times * float(moved.max()))
         err = float(np.abs(row.astype(np.float64) - want[rid][position]).max())
         assert np.isfinite(row).all() and err <= limit, (f"{what}: first wrong token is request {rid!r} position "
                                                          f"{position}: max |diff| {err:.3e} > {limit:.3e}")
+        if err > max(REL[dtype] * scale, times * usual):
+            over.append((rid, position))
+    assert len(over) <= 1 + len(got) // 20, f"{what}: {len(over)} of {len(got)} rows beyond the usual rounding, the first {over[:3]}"
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
